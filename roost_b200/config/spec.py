@@ -25,14 +25,33 @@ class NormSpec:
 
 
 @dataclass(frozen=True)
+class RotationScaling:
+    """How a rotation's frequencies f_i are stretched by ``factor`` for sequences longer than ``original`` positions.
+    ``llama3``: with the wavelength l = 2 pi / f, f stays where l < original / high, becomes f / factor where l > original / low, and
+    between the two is (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+    ``yarn``: with at(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta), the element that turns t times within ``original``
+    positions, lo = max(floor(at(fast)), 0), hi = min(ceil(at(slow)), rotary_dim - 1) and ramp_i = clamp((i - lo) / max(hi - lo,
+    0.001), 0, 1), the frequency is f_i / factor ramp_i + f_i (1 - ramp_i), and cosines and sines are multiplied by
+    0.1 ln(factor) + 1."""
+    kind: str
+    factor: float
+    original: float
+    low: float = 0.0
+    high: float = 0.0
+    fast: float = 0.0
+    slow: float = 0.0
+
+
+@dataclass(frozen=True)
 class PositionSpec:
     """Position encoding applied inside a mixer. ``rope_neox``: rotation of the first ``rotary_dim``
     elements of each head, pairs (i, i + rotary_dim/2), frequencies theta^(-2i/rotary_dim). ``rope_interleaved``: the same
-    angles with element 2i paired with element 2i + 1."""
+    angles with element 2i paired with element 2i + 1. ``scaling`` changes the frequencies (and may scale cosines and sines)."""
     kind: str = "rope_neox"
     rotary_dim: int = 0
     theta: float = 10000.0
     max_positions: int = 0
+    scaling: RotationScaling | None = None
 
 
 @dataclass(frozen=True)
@@ -84,7 +103,8 @@ class LatentAttentionSpec(MixerSpec):
 @dataclass(frozen=True)
 class SinkAttentionSpec(MixerSpec):
     """Grouped-query causal attention whose values have a size of their own (``v_dim``) and whose softmax may have a sink:
-    with ``sink`` the denominator is 1 + sum exp(s_j), a key of score 0 that has no value. Queries and keys are rotated
+    with ``sink`` the denominator is 1 + sum exp(s_j), a key of score 0 that has no value; with ``learned_sink`` too it is
+    exp(sink_h) + sum exp(s_j), sink_h a stored number a query head, taken as it is (``scale`` does not touch it). Queries and keys are rotated
     (``position``) and then, with ``unit_norm_eps`` set, divided by their root mean square over ``head_dim`` (eps inside the
     root, no weight). ``window`` counts the keys a query sees, its own included (None: every earlier key). With ``softcap``
     c > 0 a score s (already scaled) becomes c tanh(s / c). ``bias``: the q, k and v projections add a stored vector. The
@@ -97,11 +117,43 @@ class SinkAttentionSpec(MixerSpec):
     v_dim: int = 0
     scale: float = 0.0
     sink: bool = True
+    learned_sink: bool = False
     unit_norm_eps: float | None = None
     position: PositionSpec | None = None
     window: int | None = None
     softcap: float = 0.0
     bias: bool = False
+
+
+@dataclass(frozen=True)
+class TalkingAttentionSpec(MixerSpec):
+    """Grouped-query causal softmax attention whose scores are mixed across the heads first (talking heads): own_g = (q_g . k) ``scale``
+    with head g's own key/value head, score_h = sum_g T[h, g] own_g with a stored matrix T, then head h's softmax and head h's values.
+    Queries and keys are rotated (``position``); ``window`` counts the keys a query sees, its own included (None: every earlier key).
+    ``bias``: the q, k and v projections add stored vectors; ``out_bias``: the output projection too. With ``output_gate`` the heads side by
+    side are multiplied element by element by sigmoid(W_g h) before the output projection."""
+    kind: str = "talking_attention"
+    hidden: int = 0
+    num_heads: int = 0
+    num_kv_heads: int = 0
+    head_dim: int = 0
+    v_dim: int = 0
+    scale: float = 0.0
+    position: PositionSpec | None = None
+    window: int | None = None
+    bias: bool = False
+    output_gate: bool = False
+    out_bias: bool = False
+
+
+@dataclass(frozen=True)
+class MinGruSpec(MixerSpec):
+    """A recurrence a channel whose gates read only the current token (the minimal gated recurrent unit): z = sigmoid(W_z h + b_z),
+    u = W_x h + b_x, both ``width`` wide, c = u + 1/2 where u >= 0 and sigmoid(u) elsewhere; S <- (1 - z) S + z c from S = 0; the output is
+    W_o (S silu(W_g h)). S is kept per request in 32-bit."""
+    kind: str = "min_gru"
+    hidden: int = 0
+    width: int = 0
 
 
 @dataclass(frozen=True)
@@ -176,7 +228,10 @@ class RetentionSpec(MixerSpec):
     nothing divides. q = W_q h, k = W_k h (``num_heads`` x ``head_dim``),
     v = W_v h (``num_heads`` x ``v_dim``); q and k are rotated (``position``), k then multiplied by head_dim^(-1/2); per head
     S <- decay_h S + k v^T from S = 0, o = S^T q. Each head's o is divided by its root mean square (``eps``, no weight); the heads side
-    by side are multiplied by silu(W_g h) and projected out. S is kept per request in 32-bit."""
+    by side are multiplied by silu(W_g h) and projected out. S is kept per request in 32-bit.
+    Options: ``activation`` "silu" puts SiLU on q, k and v (with no rotation); ``key_scale`` replaces head_dim^(-1/2); ``norm`` "all" divides
+    the heads side by side by one root mean square instead of each by its own; ``norm_weight``: a stored weight as wide as the heads
+    multiplies the normed output; ``gate`` "sigmoid": the output gate is sigmoid(W_g h)."""
     kind: str = "retention"
     hidden: int = 0
     num_heads: int = 0
@@ -185,6 +240,11 @@ class RetentionSpec(MixerSpec):
     decay: tuple = ()
     eps: float = 1e-6
     position: PositionSpec | None = None
+    activation: str = "none"
+    key_scale: float | None = None
+    norm: str = "head"
+    norm_weight: bool = False
+    gate: str = "silu"
 
 
 @dataclass(frozen=True)
@@ -213,13 +273,15 @@ class SigmoidAttentionSpec(MixerSpec):
 
 @dataclass(frozen=True)
 class ParallelMixerSpec(MixerSpec):
-    """Several mixers side by side that read the same input; the result is the mean of their outputs, each first divided by
-    its root mean square over the model width (``eps``) and multiplied by a weight of its own. Every branch keeps the cache
-    or state its own kind asks for."""
+    """Several mixers side by side that read the same input. ``combine`` "normed_mean": the result is the mean of their outputs, each
+    first divided by its root mean square over the model width (``eps``) and multiplied by a weight of its own. "weighted_sum": the result
+    is the sum of their outputs, each times its entry of ``factors``. Every branch keeps the cache or state its own kind asks for."""
     kind: str = "parallel"
     hidden: int = 0
     branches: tuple = ()
     eps: float = 1e-6
+    combine: str = "normed_mean"
+    factors: tuple = ()
 
 
 @dataclass(frozen=True)
@@ -242,7 +304,7 @@ class GatedMlpSpec(FeedForwardSpec):
 @dataclass(frozen=True)
 class DenseMlpSpec(FeedForwardSpec):
     """down(act(x Wu^T)), no gate. ``activation`` "xielu": with two stored numbers (p, q), act(z) = softplus(p) z^2 + z / 2 for
-    z > 0 and (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0."""
+    z > 0 and (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 for z <= 0; "relu_squared": act(z) = max(z, 0)^2, nothing stored."""
     kind: str = "dense_mlp"
     hidden: int = 0
     intermediate: int = 0
@@ -366,7 +428,9 @@ class BlockSpec:
     activation dtype. ``pre_norm_wide``: the same with the stream kept and summed in 32-bit whatever the activation dtype
     is; its ``feed_forward`` and ``post_mixer_norm`` may be None (a layer that is its mixer only). ``pre_norm_streams``:
     the same two sublayers over several 32-bit residual streams, read and written through ``connection``. ``pre_norm_gated``:
-    ``pre_norm_wide`` with every sublayer's output scaled by a gate of its ``connection`` (``sigmoid_gate``) before the sum."""
+    ``pre_norm_wide`` with every sublayer's output scaled by a gate of its ``connection`` (``sigmoid_gate``) before the sum.
+    ``sandwich_wide``: ``pre_norm_wide`` with one more norm on every sublayer's output before it joins the stream (``mixer_out_norm``,
+    ``feed_forward_out_norm``)."""
     mixer: MixerSpec
     feed_forward: FeedForwardSpec | None
     input_norm: NormSpec
@@ -374,6 +438,8 @@ class BlockSpec:
     kind: str = "pre_norm"
     connection: ConnectionSpec | None = None
     token_input: TokenInputSpec | None = None     # ``pre_norm_wide`` only: added after the last sublayer
+    mixer_out_norm: NormSpec | None = None        # ``sandwich_wide`` only: the norms between a sublayer's output and the sum
+    feed_forward_out_norm: NormSpec | None = None
 
 
 @dataclass(frozen=True)

@@ -2,6 +2,7 @@
 //
 // xielu:          y = a_pos z^2 + z / 2 for z > 0, y = a_neg (exp(z) - 1 - z) + z / 2 for z <= 0, on the 32-bit value, rounded once.
 //                 Vector form: 16 bytes a thread where the pointers and the count allow.
+// relu_squared:   y = max(z, 0)^2, likewise.
 // head_gate_mul:  x[t, h, :] *= sigmoid(g[t, col + h]), one gate a token and head, in place.
 #include "common.cuh"
 
@@ -29,6 +30,32 @@ __global__ void xielu_vec_kernel(const T* __restrict__ x, T* __restrict__ out, s
   Vec<T>::load(x + i * Vec<T>::N, v);
 #pragma unroll
   for (int j = 0; j < Vec<T>::N; ++j) v[j] = xielu_f(v[j], a_pos, a_neg);
+  Vec<T>::store(out + i * Vec<T>::N, v);
+}
+
+template <typename T>
+__global__ void relu_squared_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float z = fmaxf(to_float(x[i]), 0.f);
+  out[i] = from_float<T>(z * z);
+}
+
+template <typename T>
+__global__ void relu_squared_vec_kernel(const T* __restrict__ x, T* __restrict__ out, size_t nvec) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= nvec) return;
+  float v[Vec<T>::N];
+  Vec<T>::load(x + i * Vec<T>::N, v);
+#pragma unroll
+  for (int j = 0; j < Vec<T>::N; ++j) {
+    v[j] = fmaxf(v[j], 0.f);
+    v[j] *= v[j];
+  }
   Vec<T>::store(out + i * Vec<T>::N, v);
 }
 
@@ -64,6 +91,18 @@ extern "C" int roost_xielu(const void* x, void* out, int64_t n, float a_pos, flo
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(xielu_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const T*)x, (T*)out, (size_t)n,
                                                a_pos, a_neg));
   return check_launch("xielu");
+}
+
+extern "C" int roost_relu_squared(const void* x, void* out, int64_t n, int dtype, roost_stream_t stream) {
+  ROOST_REQUIRE(n >= 0 && (n == 0 || (x && out)), "relu_squared: a pointer is null");
+  if (n == 0) return ROOST_OK;
+  const int vec = dtype == ROOST_F32 ? 4 : 8;
+  const bool whole = n % vec == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0;
+  const int64_t items = whole ? n / vec : n, blocks = (items + 255) / 256;
+  if (blocks > 2147483647LL) return fail(ROOST_ERR_UNSUPPORTED, "relu_squared: too many numbers for one launch");
+  ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(whole ? relu_squared_vec_kernel<T> : relu_squared_kernel<T>, dim3((unsigned)blocks), dim3(256), 0,
+                                               (cudaStream_t)stream, (const T*)x, (T*)out, (size_t)items));
+  return check_launch("relu_squared");
 }
 
 extern "C" int roost_head_gate_mul(void* x, const void* g, int64_t ld_g, int col, int tokens, int heads, int vdim, int dtype, roost_stream_t stream) {

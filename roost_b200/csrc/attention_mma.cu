@@ -22,6 +22,13 @@
 namespace roost {
 
 constexpr float kLog2e = 1.4426950408889634f;
+
+// The sink's term in the denominator of head h for a running maximum m (in log2 units): exp(sinks[h]) / 2^m, with the sink's
+// logit zero where there are no stored ones.
+__device__ __forceinline__ float sink_term(float sink, const float* __restrict__ sinks, int h, float m) {
+  if (sink == 0.f) return 0.f;
+  return exp2f((sinks != nullptr ? sinks[h] * kLog2e : 0.f) - m);
+}
 constexpr int kDecodeTileKeys = 16;  // keys per tile of a decode warp
 constexpr int kDecodeStages = 3;     // tiles a decode warp keeps in shared memory
 
@@ -404,7 +411,7 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
                                                                 const int32_t* __restrict__ kv_indptr,
                                                                 const int32_t* __restrict__ kv_indices, const int2* __restrict__ work,
                                                                 int q_heads, int kv_heads, int page_size, int page_shift, float scale_log2, int window,
-                                                                float cap_log2) {
+                                                                float cap_log2, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // one more term, 2^(0 - m), in every row's denominator
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -496,7 +503,7 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
     for (int r = 0; r < 2; ++r) {
       const int pr = row0 + warp * 16 * MT + mt * 16 + (lane >> 2) + r * 8;
       if (pr >= rows_total) continue;
-      const float lr = st.l[mt][r] + sink * exp2f(-(st.m[mt][r] == -INFINITY ? 0.f : st.m[mt][r]));
+      const float lr = st.l[mt][r] + sink_term(sink, sinks, kvh * group + pr % group, st.m[mt][r] == -INFINITY ? 0.f : st.m[mt][r]);
       const float inv = lr > 0.f ? 1.0f / lr : 0.f;
       __nv_bfloat16* dst = out + ((size_t)(q_start + pr / group) * q_heads + kvh * group + pr % group) * D + (lane & 3) * 2;
 #pragma unroll
@@ -521,7 +528,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
                             const int32_t* __restrict__ kv_lens, const int32_t* __restrict__ kv_indptr,
                             const int32_t* __restrict__ kv_indices, const int4* __restrict__ work, float* __restrict__ part_o,
                             float* __restrict__ part_ml, int q_heads, int kv_heads, int page_size, int page_shift, float scale_log2, int window,
-                            int slot_limit) {
+                            int slot_limit, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // added where a row's result is final, never to a partial one
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -646,7 +653,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
       o += sm_o[((size_t)ww * 16 + row) * D + col] * f;
     }
     if (slot < 0) {
-      l += sink * exp2f(-msafe);
+      l += sink_term(sink, sinks, kvh * group + row % group, msafe);
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       out[((size_t)(q_start + row / group) * q_heads + kvh * group + row % group) * D + col] = __float2bfloat16_rn(o * inv);
     } else {
@@ -729,7 +736,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
                                 const int32_t* __restrict__ q_indptr, const int32_t* __restrict__ kv_lens,
                                 const int32_t* __restrict__ kv_indptr, const int32_t* __restrict__ kv_indices,
                                 const int4* __restrict__ work, int items, float* __restrict__ part_o, float* __restrict__ part_ml, int q_heads,
-                                int kv_heads, int page_size, float scale_log2, int window, int cluster_chunks) {
+                                int kv_heads, int page_size, float scale_log2, int window, int cluster_chunks, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // added where a row's result is final, never to a partial one
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -1069,7 +1076,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
             cl_o[16 * D + row * 2 + 1] = l;
           }
         } else if (c.slot < 0) {
-          l += sink * exp2f(-msafe);
+          l += sink_term(sink, sinks, c.kvh * group + row % group, msafe);
           const float inv = l > 0.f ? 1.0f / l : 0.f;
           out[((size_t)(c.q_start + row / group) * q_heads + c.kvh * group + row % group) * D + col] = __float2bfloat16_rn(o * inv);
         } else {
@@ -1125,7 +1132,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
             o += po[cc] * f;
           }
         }
-        l += sink * exp2f(-msafe);
+        l += sink_term(sink, sinks, cl_kvh * group + row % group, msafe);
         const float inv = l > 0.f ? 1.0f / l : 0.f;
         out[((size_t)(cl_q_start + row / group) * q_heads + cl_kvh * group + row % group) * D + col] = __float2bfloat16_rn(o * inv);
       }
@@ -1150,7 +1157,8 @@ constexpr int kMergeAhead = 9;  // chunks whose partial results a merge thread l
 // merge_work[i] = (batch row, first partial slot, number of chunks | packed rows << 24, the row's first token)
 template <int D>
 __global__ void attention_merge_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                       const int4* __restrict__ merge_work, int q_heads, int kv_heads, int slot_limit, float sink) {
+                                       const int4* __restrict__ merge_work, int q_heads, int kv_heads, int slot_limit, float sink,
+                                       const float* __restrict__ sinks) {
   pdl_launch_dependents(5);
   const int4 w = merge_work[blockIdx.x];  // the step's work lists are on the device before the step's first kernel runs
   const int b = w.x, slot0 = w.y, chunks = w.z & 0xffffff, rows_total = w.z >> 24, q_start = w.w;
@@ -1205,7 +1213,7 @@ __global__ void attention_merge_kernel(__nv_bfloat16* __restrict__ out, const fl
           for (int j = 0; j < (D + 127) / 128; ++j) o[j] += po[j][c] * f;
         }
       }
-      l += sink * exp2f(-msafe);
+      l += sink_term(sink, sinks, kvh * group + row % group, msafe);
       const float inv = l > 0.f ? 1.0f / l : 0.f;
 #pragma unroll
       for (int j = 0; j < (D + 127) / 128; ++j) {
@@ -1227,7 +1235,7 @@ __global__ void attention_merge_kernel(__nv_bfloat16* __restrict__ out, const fl
         l += part_ml[pr * 2 + 1] * f;
         o += part_o[pr * D + col] * f;
       }
-      l += sink * exp2f(-msafe);
+      l += sink_term(sink, sinks, kvh * group + row % group, msafe);
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       out[out_at + col] = __float2bfloat16_rn(o * inv);
     }
@@ -1263,7 +1271,7 @@ constexpr int kPrefillTwoGroupsMinRows = 49152;
 template <int D, int MT>
 static int launch_prefill(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                           const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, int q_heads, int kv_heads,
-                          int page_size, float scale, int window, cudaStream_t s, float softcap = 0.f) {
+                          int page_size, float scale, int window, cudaStream_t s, float softcap = 0.f, const float* sinks = nullptr) {
   const size_t smem = (size_t)(64 * MT + 4 * 64) * D * 2;
   auto kernel = attention_prefill_kernel<D, MT>;
   static bool attr_set = false;  // once per process: nothing but launches happens on later calls (stream capture)
@@ -1273,7 +1281,7 @@ static int launch_prefill(const void* q, void* out, const void* k_pool, const vo
   }
   launch_kernel(kernel, dim3(items, kv_heads), dim3(128), smem, s, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_pool,
                 (const __nv_bfloat16*)v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, (const int2*)work, q_heads, kv_heads, page_size,
-                page_shift_of(page_size), scale * kLog2e, window, softcap * kLog2e);
+                page_shift_of(page_size), scale * kLog2e, window, softcap * kLog2e, sinks);
   return check_launch("attention_prefill");
 }
 
@@ -1310,7 +1318,7 @@ template <int D>
 static int launch_decode_tma(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                              const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, float* part_o,
                              float* part_ml, int q_heads, int kv_heads, int page_size, long long pool_pages, float scale, int window,
-                             cudaStream_t s, int cluster_chunks) {
+                             cudaStream_t s, int cluster_chunks, const float* sinks) {
   CUtensorMap map;
   const int box_rows = page_size < kTmaTileKeys ? page_size : kTmaTileKeys;
   const int rc = make_pool_map(&map, k_pool, v_pool, pool_pages * kv_heads * page_size, D, box_rows);
@@ -1331,7 +1339,7 @@ static int launch_decode_tma(const void* q, void* out, const void* k_pool, const
   auto kernel = box_rows == 16 ? attention_decode_tma_kernel<D, 16> : attention_decode_tma_kernel<D, 32>;
   launch_kernel_cluster(kernel, dim3(grid), dim3((kTmaConsumers + 1) * 32), smem, s, cluster_chunks > 0 ? cluster_chunks : 1, map,
                         (const __nv_bfloat16*)q, (__nv_bfloat16*)out, q_indptr, kv_lens, kv_indptr, kv_indices, (const int4*)work, items, part_o,
-                        part_ml, q_heads, kv_heads, page_size, scale * kLog2e, window, cluster_chunks);
+                        part_ml, q_heads, kv_heads, page_size, scale * kLog2e, window, cluster_chunks, sinks);
   return check_launch("attention_decode_tma");
 }
 
@@ -1339,13 +1347,14 @@ template <int D>
 static int launch_decode(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                          const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, const int32_t* merge_work,
                          int merge_items, int merge_rows, float* part_o, float* part_ml, int q_heads, int kv_heads, int page_size,
-                         long long pool_pages, float scale, int window, cudaStream_t s, int slot_limit = kNoSlotLimit) {
+                         long long pool_pages, float scale, int window, cudaStream_t s, int slot_limit = kNoSlotLimit,
+                         const float* sinks = nullptr) {
   int rc = ROOST_OK;
   bool launched = false;
   if constexpr (D == 64 || D == 128) {
     if (slot_limit == kNoSlotLimit && decode_tma_serves(D, page_size, pool_pages, kv_heads, k_pool, v_pool)) {
       rc = launch_decode_tma<D>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, part_o, part_ml, q_heads,
-                                kv_heads, page_size, pool_pages, scale, window, s, 0);
+                                kv_heads, page_size, pool_pages, scale, window, s, 0, sinks);
       launched = true;
     }
   }
@@ -1362,14 +1371,14 @@ static int launch_decode(const void* q, void* out, const void* k_pool, const voi
     }
     launch_kernel(kernel, dim3(items, kv_heads), dim3(NW * 32), smem, s, (const __nv_bfloat16*)q, (__nv_bfloat16*)out,
                   (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, (const int4*)work, part_o,
-                  part_ml, q_heads, kv_heads, page_size, page_shift_of(page_size), scale * kLog2e, window, slot_limit);
+                  part_ml, q_heads, kv_heads, page_size, page_shift_of(page_size), scale * kLog2e, window, slot_limit, sinks);
     rc = check_launch("attention_decode");
   }
   if (rc != ROOST_OK || merge_items == 0) return rc;
   const int rows = merge_rows < 1 ? 1 : (merge_rows > 16 ? 16 : merge_rows);  // blocks along z; each walks the rows beyond
   launch_kernel(attention_merge_kernel<D>, dim3(merge_items, kv_heads, rows), dim3(D < 128 ? D : 128), 0, s, (__nv_bfloat16*)out,
                 (const float*)part_o, (const float*)part_ml, (const int4*)merge_work, q_heads, kv_heads, slot_limit,
-                (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f);
+                (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f, sinks);
   return check_launch("attention_merge");
 }
 
@@ -1441,7 +1450,7 @@ extern "C" int roost_attention_mma_supported(int head_dim) {
 static int attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                              const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items,
                              int tile_rows, int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                             float softcap, roost_stream_t stream) {
+                             float softcap, const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_prefill: sizes must be positive");
   ROOST_REQUIRE(tile_rows == 64 || ((tile_rows == 128 || tile_rows == 256) && head_dim <= 128),
                 "attention_prefill: a work item has 64 packed rows, or 128 or 256 up to head size 128");
@@ -1449,32 +1458,34 @@ static int attention_prefill(const void* q, long long tokens, void* out, const v
   if (kv_heads > 65535) return fail(ROOST_ERR_UNSUPPORTED, "attention_prefill: more than 65535 key/value heads");
   if (items == 0) return ROOST_OK;
   ROOST_REQUIRE(softcap >= 0.f && (softcap == 0.f || tile_rows != 256), "attention_prefill: a cap on the scores is served by the mma.sync kernels (items of 64 or 128 packed rows)");
-  if ((tile_rows == 128 || tile_rows == 256) && tokens > 0 && !(window & ROOST_ATTENTION_WIDE_WEIGHTS) && softcap == 0.f &&
+  if ((tile_rows == 128 || tile_rows == 256) && tokens > 0 && !(window & ROOST_ATTENTION_WIDE_WEIGHTS) && softcap == 0.f && sinks == nullptr &&
       prefill_tc_serves(head_dim, q_heads, kv_heads, page_size, pool_pages, k_pool, v_pool, q)) {
     return launch_prefill_tc(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads,
                              head_dim, page_size, pool_pages, scale, window, (cudaStream_t)stream);
   }
-  ROOST_REQUIRE(tile_rows != 256 || !(window & ROOST_ATTENTION_WIDE_WEIGHTS), "attention_prefill: work items of 256 packed rows belong to the tcgen05 kernel, which takes no wide weights");
+  ROOST_REQUIRE(tile_rows != 256 || (!(window & ROOST_ATTENTION_WIDE_WEIGHTS) && sinks == nullptr),
+                "attention_prefill: work items of 256 packed rows belong to the tcgen05 kernel, which takes no wide weights and no stored sinks");
   if (tile_rows == 128) {
     switch (head_dim) {
-      case 16: return launch_prefill<16, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap);
-      case 32: return launch_prefill<32, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap);
-      case 64: return launch_prefill<64, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap);
-      case 128: return launch_prefill<128, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap);
+      case 16: return launch_prefill<16, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
+      case 32: return launch_prefill<32, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
+      case 64: return launch_prefill<64, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
+      case 128: return launch_prefill<128, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
       default: return fail(ROOST_ERR_UNSUPPORTED, "attention_prefill: no tensor-core kernel for this head size");
     }
   }
   ROOST_DISPATCH_HEAD_DIM(head_dim, D, return launch_prefill<D, 1>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items,
-                                                                    q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap));
+                                                                    q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks));
   return ROOST_OK;
 }
 
 extern "C" int roost_attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool,
                                        const int32_t* q_indptr, const int32_t* kv_lens, const int32_t* kv_indptr,
                                        const int32_t* kv_indices, const int32_t* work, int items, int tile_rows, int q_heads, int kv_heads,
-                                       int head_dim, int page_size, long long pool_pages, float scale, int window, roost_stream_t stream) {
+                                       int head_dim, int page_size, long long pool_pages, float scale, int window, const float* sinks,
+                                       roost_stream_t stream) {
   return attention_prefill(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads, head_dim,
-                           page_size, pool_pages, scale, window, 0.f, stream);
+                           page_size, pool_pages, scale, window, 0.f, sinks, stream);
 }
 
 // The same with a cap c on the scores: a score s (scaled) becomes c tanh(s / c) before the mask and the softmax. mma.sync kernels only.
@@ -1482,16 +1493,16 @@ extern "C" int roost_attention_prefill_capped(const void* q, long long tokens, v
                                               const int32_t* q_indptr, const int32_t* kv_lens, const int32_t* kv_indptr,
                                               const int32_t* kv_indices, const int32_t* work, int items, int tile_rows, int q_heads,
                                               int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                                              float softcap, roost_stream_t stream) {
+                                              float softcap, const float* sinks, roost_stream_t stream) {
   return attention_prefill(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads, head_dim,
-                           page_size, pool_pages, scale, window, softcap, stream);
+                           page_size, pool_pages, scale, window, softcap, sinks, stream);
 }
 
 extern "C" int roost_attention_decode(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                       const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                                       int items, const int32_t* merge_work, int merge_items, int merge_rows, float* part_o, float* part_ml,
                                       int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                                      roost_stream_t stream) {
+                                      const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && merge_items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_decode: sizes must be positive");
   ROOST_REQUIRE(q_heads % kv_heads == 0, "attention_decode: q_heads must be a multiple of kv_heads");
   ROOST_REQUIRE(merge_items == 0 || (part_o && part_ml && merge_work), "attention_decode: the workspace for split rows is missing");
@@ -1499,7 +1510,7 @@ extern "C" int roost_attention_decode(const void* q, void* out, const void* k_po
   if (items == 0) return ROOST_OK;
   ROOST_DISPATCH_HEAD_DIM(head_dim, D, return launch_decode<D>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items,
                                                                 merge_work, merge_items, merge_rows, part_o, part_ml, q_heads, kv_heads,
-                                                                page_size, pool_pages, scale, window, (cudaStream_t)stream));
+                                                                page_size, pool_pages, scale, window, (cudaStream_t)stream, kNoSlotLimit, sinks));
   return ROOST_OK;
 }
 
@@ -1522,7 +1533,8 @@ extern "C" int roost_attention_decode_cluster_supported(int head_dim, int page_s
 extern "C" int roost_attention_decode_cluster(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                               const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices,
                                               const int32_t* work, int items, int cluster_chunks, int q_heads, int kv_heads, int head_dim,
-                                              int page_size, long long pool_pages, float scale, int window, roost_stream_t stream) {
+                                              int page_size, long long pool_pages, float scale, int window, const float* sinks,
+                                              roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_decode_cluster: sizes must be positive");
   ROOST_REQUIRE(q_heads % kv_heads == 0, "attention_decode_cluster: q_heads must be a multiple of kv_heads");
   ROOST_REQUIRE(cluster_chunks == 1 || cluster_chunks == 2 || cluster_chunks == 4 || cluster_chunks == 8,
@@ -1536,10 +1548,10 @@ extern "C" int roost_attention_decode_cluster(const void* q, void* out, const vo
   const cudaStream_t s = (cudaStream_t)stream;
   if (head_dim == 64) {
     return launch_decode_tma<64>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, nullptr, nullptr, q_heads,
-                                 kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks);
+                                 kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks, sinks);
   }
   return launch_decode_tma<128>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, nullptr, nullptr, q_heads,
-                                kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks);
+                                kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks, sinks);
 }
 
 constexpr size_t kStaticScratchFloats = 4u * 1024u * 1024u;  // 16 MiB

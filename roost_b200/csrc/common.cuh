@@ -113,7 +113,8 @@ __device__ __forceinline__ float gate_fn(float g, float u, int act, float limit)
   return g / (1.0f + expf(-g)) * u;
 }
 
-// exp(x) for x <= 0 to about one unit in the last place: x = j ln2 + r with ln2 in two parts, a degree-7 polynomial in r.
+// exp(x) for x <= 0 to about one unit in the last place: x = j ln2 + r with ln2 in two parts, a degree-7 polynomial in r (the method
+// and the coefficients of expf in the Cephes Mathematical Library, Stephen L. Moshier).
 __device__ __forceinline__ float exp_nearest(float x) {
   if (x < -87.0f) return 0.f;
   const float j = rintf(x * 1.44269504088896341f);
@@ -128,6 +129,9 @@ __device__ __forceinline__ float exp_nearest(float x) {
   const float y = fmaf(p * r, r, r) + 1.0f;
   return y * __int_as_float(((int)j + 127) << 23);
 }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 
 __device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 

@@ -77,8 +77,6 @@ __device__ __forceinline__ void store_row32<float>(float* dst, const uint32_t (&
   }
 }
 
-__device__ __forceinline__ float silu_f(float g) { return g / (1.0f + expf(-g)); }
-
 // EPI 0: out = acc. EPI 1 (SwiGLU): w's rows come in blocks of 256, 128 gate rows followed by the 128 up rows of the same
 // outputs, so a tile's columns 0..127 are gate and 128..255 the matching up values: out[m, n0/2 + j] = silu(gate_j) * up_j,
 // and out has n/2 columns.

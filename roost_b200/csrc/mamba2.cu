@@ -17,8 +17,6 @@
 
 namespace roost {
 
-__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
-
 template <typename T>
 __global__ void mamba2_conv_kernel(const T* __restrict__ u, int64_t ld, int col, T* __restrict__ out, const float* __restrict__ w,
                                    const float* __restrict__ bias, const float* __restrict__ state, int64_t state_stride, int conv_off,

@@ -18,7 +18,7 @@
 // memory in its place, and a second walk of every chunk from there writes the outputs and, from a row's last chunk, the slot.
 //
 // head_norm_gate: per token and head, o / sqrt(mean(o^2) + eps) * w * sigmoid(g) (w may be absent; with gate_silu the gate is
-// g sigmoid(g)), rounded once.
+// g sigmoid(g)), rounded once. One head as wide as the row takes a block a token instead of a warp a head.
 #include "common.cuh"
 
 namespace roost {
@@ -251,6 +251,25 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const T* __re
   }
 }
 
+template <typename T>
+__global__ void row_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ u, int64_t ld_u, int col, const float* __restrict__ w,
+                                     T* __restrict__ out, int width, float eps, int gate_silu) {
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  const float* x = o + t * width;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
+  ss = block_sum(ss, scratch);
+  const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float g = to_float(u[t * ld_u + col + i]);
+    const float y = x[i] * inv * (w != nullptr ? w[i] : 1.0f) / (1.0f + expf(-g));
+    out[t * width + i] = from_float<T>(gate_silu ? y * g : y);
+  }
+}
+
 }  // namespace roost
 
 using namespace roost;
@@ -308,6 +327,12 @@ extern "C" int roost_head_norm_gate(const float* o, const void* u, int64_t ld_u,
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && vdim > 0 && eps > 0.f && col >= 0 && ld_u >= col + (int64_t)heads * vdim, "head_norm_gate: sizes do not fit");
   ROOST_REQUIRE(o && u && out, "head_norm_gate: a pointer is null");
   if (tokens == 0) return ROOST_OK;
+  if (heads == 1) {
+    const int threads = vdim >= 1024 ? 512 : (vdim >= 256 ? 256 : 64);
+    ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(row_norm_gate_kernel<T>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, o, (const T*)u, ld_u, col, w,
+                                                 (T*)out, vdim, eps, gate_silu));
+    return check_launch("head_norm_gate");
+  }
   const int threads = heads >= 8 ? 256 : (heads >= 4 ? 128 : 32 * heads);
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(head_norm_gate_kernel<T>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, o, (const T*)u, ld_u, col,
                                                w, (T*)out, heads, vdim, eps, gate_silu));

@@ -11,7 +11,8 @@
 //
 // scan: one warp (a block) per (row, head, 32 columns of S). A lane keeps its column of S in registers (dim up to 128) or in
 // shared memory (beyond); a token's (k, q) are staged in shared memory once and read by all lanes; the next token's inputs are
-// loaded while the current one is multiplied.
+// loaded while the current one is multiplied. Where nothing is rotated the scan reads the projection's row [q heads | k heads | v heads]
+// itself (RAW): q, k and v pass SiLU (act 1) or stay as they are, k is multiplied by k_scale, all in 32-bit, and no prepare kernel runs.
 //
 // Steps of many tokens cut every row into chunks of 64 tokens that run side by side (three launches): a chunk of n tokens walked
 // from S = 0 ends with S'; a state S before the chunk is decay^n S + S' after it. The first walk leaves every chunk's own S', one
@@ -75,8 +76,9 @@ __device__ __forceinline__ bool retention_chunk_of_block(const int32_t* __restri
 // MODE 0: a warp walks its row's tokens from the slot and writes the slot back. MODE 1: a warp walks one chunk from S = 0 and
 // leaves S' in ws[chunk]; a row's last chunk is skipped. MODE 2: a warp walks one chunk from ws[chunk] (the carry kernel put the
 // chunk's true starting state there) and writes the outputs; a row's last chunk writes the slot.
-template <typename T, int DREG, int MODE>
-__global__ void __launch_bounds__(32) retention_scan_kernel(const float* __restrict__ qk, const T* __restrict__ v, int64_t ldv,
+template <typename T, int DREG, int MODE, bool RAW>
+__global__ void __launch_bounds__(32) retention_scan_kernel(const void* __restrict__ qk_rows, int64_t ldqk, int act, float k_scale,
+                                                           const T* __restrict__ v, int64_t ldv,
                                                            float* __restrict__ out, float* state, int64_t state_stride,
                                                            const float* __restrict__ decay, const int32_t* __restrict__ q_indptr,
                                                            const int32_t* __restrict__ slots, int rows, int heads, int dim, int vdim, float* ws) {
@@ -115,12 +117,22 @@ __global__ void __launch_bounds__(32) retention_scan_kernel(const float* __restr
   // the next token's inputs, loaded one token ahead
   float nk[NN], nq[NN], nv;
   auto load = [&](int t) {
-    const float* row = qk + (size_t)t * 2 * QK;
+    if constexpr (RAW) {
+      const T* row = reinterpret_cast<const T*>(qk_rows) + (size_t)t * ldqk;
 #pragma unroll
-    for (int i = 0; i < NN; ++i) {
-      const int d = lane + 32 * i;
-      nq[i] = d < dim ? row[(size_t)h * dim + d] : 0.f;
-      nk[i] = d < dim ? row[QK + (size_t)h * dim + d] : 0.f;
+      for (int i = 0; i < NN; ++i) {
+        const int d = lane + 32 * i;
+        nq[i] = d < dim ? to_float(row[(size_t)h * dim + d]) : 0.f;
+        nk[i] = d < dim ? to_float(row[QK + (size_t)h * dim + d]) : 0.f;
+      }
+    } else {
+      const float* row = reinterpret_cast<const float*>(qk_rows) + (size_t)t * 2 * QK;
+#pragma unroll
+      for (int i = 0; i < NN; ++i) {
+        const int d = lane + 32 * i;
+        nq[i] = d < dim ? row[(size_t)h * dim + d] : 0.f;
+        nk[i] = d < dim ? row[QK + (size_t)h * dim + d] : 0.f;
+      }
     }
     nv = live ? to_float(v[(size_t)t * ldv + (size_t)h * vdim + col]) : 0.f;
   };
@@ -130,9 +142,9 @@ __global__ void __launch_bounds__(32) retention_scan_kernel(const float* __restr
 #pragma unroll
     for (int i = 0; i < NN; ++i) {
       const int d = lane + 32 * i;
-      if (d < dim) stage[d] = make_float2(nk[i], nq[i]);
+      if (d < dim) stage[d] = !RAW ? make_float2(nk[i], nq[i]) : (act ? make_float2(silu_f(nk[i]) * k_scale, silu_f(nq[i])) : make_float2(nk[i] * k_scale, nq[i]));
     }
-    const float val = nv;
+    const float val = RAW && act ? silu_f(nv) : nv;
     if (t + 1 < end) load(t + 1);
     __syncwarp();
     float num = 0.f;
@@ -224,6 +236,44 @@ extern "C" int roost_retention_prepare(const void* u, int64_t ld, float* qk, con
 
 extern "C" int roost_retention_scan_chunks(int tokens, int rows) { return (tokens + kRtChunkTokens - 1) / kRtChunkTokens + rows; }
 
+namespace roost {
+
+template <typename T, bool RAW>
+static int retention_scan_launch(const void* qk, int64_t ldqk, int act, float k_scale, const T* v, int64_t ldv, float* out, float* state,
+                                 int64_t state_stride, const float* decay, const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads,
+                                 int dim, int vdim, float* ws, cudaStream_t s) {
+  const int slices = (vdim + 31) / 32;
+  const size_t stage = (size_t)4 * dim * sizeof(float);
+  const int chunks = roost_retention_scan_chunks(tokens, rows);
+#define ROOST_RT_LAUNCH(DREG, MODE, SMEM, GX)                                                                                                      \
+  do {                                                                                                                                             \
+    auto kernel = retention_scan_kernel<T, DREG, MODE, RAW>;                                                                                       \
+    if ((SMEM) > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(SMEM));                                \
+    launch_kernel(kernel, dim3((GX), heads, slices), dim3(32), (SMEM), s, qk, ldqk, act, k_scale, v, ldv, out, state, state_stride, decay,         \
+                  q_indptr, slots, rows, heads, dim, vdim, ws);                                                                                    \
+  } while (0)
+#define ROOST_RT_SCAN(DREG, SMEM)                                                                                                                  \
+  do {                                                                                                                                             \
+    if (ws == nullptr) {                                                                                                                           \
+      ROOST_RT_LAUNCH(DREG, 0, SMEM, rows);                                                                                                        \
+    } else {                                                                                                                                       \
+      ROOST_RT_LAUNCH(DREG, 1, SMEM, chunks);                                                                                                      \
+      launch_kernel(retention_carry_kernel, dim3(rows, heads, (dim * vdim + 255) / 256), dim3(256), 0, s, (const float*)state, state_stride, ws,   \
+                    decay, q_indptr, slots, heads, dim, vdim);                                                                                     \
+      ROOST_RT_LAUNCH(DREG, 2, SMEM, chunks);                                                                                                      \
+    }                                                                                                                                              \
+  } while (0)
+  if (dim <= 32) ROOST_RT_SCAN(32, stage);
+  else if (dim <= 64) ROOST_RT_SCAN(64, stage);
+  else if (dim <= 128) ROOST_RT_SCAN(128, stage);
+  else ROOST_RT_SCAN(0, stage + (size_t)dim * 32 * sizeof(float));
+#undef ROOST_RT_SCAN
+#undef ROOST_RT_LAUNCH
+  return check_launch("retention_scan");
+}
+
+}  // namespace roost
+
 // ws (float[chunks * heads * dim * vdim], chunks = roost_retention_scan_chunks(tokens, rows)): rows are cut into chunks that run side
 // by side (three launches); null: every row is walked in one pass.
 extern "C" int roost_retention_scan(const float* qk, const void* v, int64_t ldv, float* out, float* state, int64_t state_stride, const float* decay,
@@ -233,37 +283,25 @@ extern "C" int roost_retention_scan(const float* qk, const void* v, int64_t ldv,
   ROOST_REQUIRE(qk && v && out && state && decay && q_indptr && slots, "retention_scan: a pointer is null");
   ROOST_REQUIRE(ldv >= (int64_t)heads * vdim && state_stride >= (int64_t)heads * dim * vdim, "retention_scan: a row or a slot is too narrow");
   if (dim > 1024) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan: heads of more than 1024 keys");
-  const int slices = (vdim + 31) / 32;
-  if (heads > 65535 || slices > 65535) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan: too many heads or values");
+  if (heads > 65535 || (vdim + 31) / 32 > 65535) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan: too many heads or values");
   if (rows == 0 || tokens == 0) return ROOST_OK;
-  cudaStream_t s = (cudaStream_t)stream;
-  const size_t stage = (size_t)4 * dim * sizeof(float);
-  const int chunks = roost_retention_scan_chunks(tokens, rows);
-#define ROOST_RT_LAUNCH(DREG, MODE, SMEM, GX)                                                                                                     \
-  do {                                                                                                                                            \
-    auto kernel = retention_scan_kernel<T, DREG, MODE>;                                                                                           \
-    if ((SMEM) > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(SMEM));                               \
-    launch_kernel(kernel, dim3((GX), heads, slices), dim3(32), (SMEM), s, qk, (const T*)v, ldv, out, state, state_stride, decay, q_indptr, slots, \
-                  rows, heads, dim, vdim, ws);                                                                                                    \
-  } while (0)
-#define ROOST_RT_SCAN(DREG, SMEM)                                                                                                                 \
-  do {                                                                                                                                            \
-    if (ws == nullptr) {                                                                                                                          \
-      ROOST_RT_LAUNCH(DREG, 0, SMEM, rows);                                                                                                       \
-    } else {                                                                                                                                      \
-      ROOST_RT_LAUNCH(DREG, 1, SMEM, chunks);                                                                                                     \
-      launch_kernel(retention_carry_kernel, dim3(rows, heads, (dim * vdim + 255) / 256), dim3(256), 0, s, (const float*)state, state_stride, ws,  \
-                    decay, q_indptr, slots, heads, dim, vdim);                                                                                    \
-      ROOST_RT_LAUNCH(DREG, 2, SMEM, chunks);                                                                                                     \
-    }                                                                                                                                             \
-  } while (0)
-  ROOST_DISPATCH_DTYPE(dtype, T, {
-    if (dim <= 32) ROOST_RT_SCAN(32, stage);
-    else if (dim <= 64) ROOST_RT_SCAN(64, stage);
-    else if (dim <= 128) ROOST_RT_SCAN(128, stage);
-    else ROOST_RT_SCAN(0, stage + (size_t)dim * 32 * sizeof(float));
-  });
-#undef ROOST_RT_SCAN
-#undef ROOST_RT_LAUNCH
-  return check_launch("retention_scan");
+  ROOST_DISPATCH_DTYPE(dtype, T, return (retention_scan_launch<T, false>(qk, 0, 0, 1.0f, (const T*)v, ldv, out, state, state_stride, decay, q_indptr, slots,
+                                                                         rows, tokens, heads, dim, vdim, ws, (cudaStream_t)stream)));
+}
+
+// The same over the projection's rows u = [q heads | k heads | v heads | ...], ld apart, where nothing is rotated: act 1 puts SiLU on q, k
+// and v; the keys are multiplied by k_scale.
+extern "C" int roost_retention_scan_raw(const void* u, int64_t ld, int act, float k_scale, float* out, float* state, int64_t state_stride,
+                                        const float* decay, const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim,
+                                        int vdim, float* ws, int dtype, roost_stream_t stream) {
+  ROOST_REQUIRE(rows >= 0 && tokens >= 0 && heads > 0 && dim > 0 && vdim > 0, "retention_scan_raw: sizes must be positive");
+  ROOST_REQUIRE(u && out && state && decay && q_indptr && slots, "retention_scan_raw: a pointer is null");
+  ROOST_REQUIRE(act == 0 || act == 1, "retention_scan_raw: the activation is none (0) or SiLU (1)");
+  ROOST_REQUIRE(ld >= (int64_t)heads * (2 * dim + vdim) && state_stride >= (int64_t)heads * dim * vdim, "retention_scan_raw: a row or a slot is too narrow");
+  if (dim > 1024) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan_raw: heads of more than 1024 keys");
+  if (heads > 65535 || (vdim + 31) / 32 > 65535) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan_raw: too many heads or values");
+  if (rows == 0 || tokens == 0) return ROOST_OK;
+  ROOST_DISPATCH_DTYPE(dtype, T, return (retention_scan_launch<T, true>(u, ld, act, k_scale, (const T*)u + (size_t)2 * heads * dim, ld, out, state,
+                                                                        state_stride, decay, q_indptr, slots, rows, tokens, heads, dim, vdim, ws,
+                                                                        (cudaStream_t)stream)));
 }

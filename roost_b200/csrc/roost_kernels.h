@@ -17,7 +17,7 @@
 extern "C" {
 #endif
 
-#define ROOST_ABI_VERSION 15
+#define ROOST_ABI_VERSION 16
 
 #define ROOST_OK 0
 #define ROOST_ERR_INVALID 1      /* an argument is out of range or inconsistent; nothing was launched */
@@ -34,7 +34,8 @@ extern "C" {
 #define ROOST_ACT_CLAMPED_SWISH 2
 
 /* Added to the `window` argument of the tensor-core attention entry points (roost_attention_prefill, _decode, _decode_cluster,
- * _decode_static): the softmax's denominator gets one more term, exp(0 - maximum), a key of score 0 that has no value. */
+ * _decode_static): the softmax's denominator gets one more term, exp(0 - maximum), a key of score 0 that has no value. Where the
+ * entry point's `sinks` (float, one a query head) is not null the term is exp(sinks[h] - maximum) instead. */
 #define ROOST_ATTENTION_SINK (1 << 30)
 /* Also added to `window`: the softmax weights enter the second product as two bfloat16 operands, their rounding and what it left
  * over, so that 16 bits of the 32-bit weights count (the denominator is summed from the 32-bit weights anyway). The mma.sync
@@ -132,18 +133,18 @@ void roost_attention_set_prefill_tc(int on);
 int roost_attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                             const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                             int items, int tile_rows, int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages,
-                            float scale, int window, roost_stream_t stream);
+                            float scale, int window, const float* sinks, roost_stream_t stream);
 /* The same with a cap c on the scores: a scaled score s becomes c tanh(s / c) before the mask and the softmax. Served by the mma.sync
  * kernels: items of 64 or 128 packed rows (roost_attention_prefill_tile_rows_mma). */
 int roost_attention_prefill_capped(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                             const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                             int items, int tile_rows, int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages,
-                            float scale, int window, float softcap, roost_stream_t stream);
+                            float scale, int window, float softcap, const float* sinks, roost_stream_t stream);
 int roost_attention_decode(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                            const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                            int items, const int32_t* merge_work, int merge_items, int merge_rows, float* part_o, float* part_ml,
                            int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                           roost_stream_t stream);
+                           const float* sinks, roost_stream_t stream);
 void roost_attention_set_decode_tma(int on);
 int roost_attention_status(void);
 /* The split decode attention without partial results in memory and without a merge kernel: the grid is thread-block
@@ -158,7 +159,7 @@ int roost_attention_decode_cluster_supported(int head_dim, int page_size, long l
 int roost_attention_decode_cluster(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                    const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                                    int items, int cluster_chunks, int q_heads, int kv_heads, int head_dim, int page_size,
-                                   long long pool_pages, float scale, int window, roost_stream_t stream);
+                                   long long pool_pages, float scale, int window, const float* sinks, roost_stream_t stream);
 
 /* The split decode attention without a workspace argument. It has no counterpart in the reference: it exists for
  * callers that must not allocate device memory while they run (a host that gave the whole GPU to its own arena at
@@ -375,14 +376,15 @@ int roost_gated_act_mul(const void* x, void* out, int tokens, int inter, int blo
  * entry from k_base and v_base. */
 int roost_sink_attention_prepare(void* qkv, int64_t ld, void* q_out, void* k_base, void* v_base, int entry, const double* inv_freq,
                                  const int32_t* positions, const int32_t* slot_mapping, int tokens, int heads, int kv_heads, int dim, int vdim,
-                                 int rot_dims, float eps, int page_size, int halves, int dtype, roost_stream_t stream);
-/* out [tokens, heads * vdim]. sink != 0: one is added to the softmax's denominator. splits > 1: a token's key tiles of 32 are
+                                 int rot_dims, float eps, int page_size, int halves, float amplitude, int dtype, roost_stream_t stream);
+/* out [tokens, heads * vdim]. sink != 0: exp(sinks[h]) is added to the softmax's denominator (one where sinks is null). splits > 1: a token's key tiles of 32 are
  * dealt in ranges of tiles_per_split to `splits` blocks whose partials (part: float[tokens * heads * splits * (vdim + 2)]) a
  * second kernel combines. */
 int roost_sink_attention(const void* qkv, int64_t ld, void* out, float* part, const void* k_base, const void* v_base, int entry,
                          const int32_t* positions, const int32_t* token_row, const int32_t* kv_indptr, const int32_t* kv_indices, int tokens,
                          int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink, int splits, int tiles_per_split,
-                         int window, float softcap, int dtype, roost_stream_t stream);   /* window 0: every earlier key; softcap 0: none */
+                         int window, float softcap, const float* sinks, int dtype, roost_stream_t stream);   /* window 0: every earlier
+                                                                                                 key; softcap 0: none */
 
 /* ---- the Mamba selective scan (mamba1.cu) ---- */
 /* Per (row, channel): dt = softplus(dt_raw + dt_bias); S <- exp(dt a_neg) S + dt x B; y = S . C + d_skip x; out = y silu(z). xc
@@ -404,10 +406,16 @@ int roost_wide_rms_norm(float* stream, const void* addend, const float* extra, c
 /* The same with the addend multiplied element by element by sigmoid(gate + gate_bias) first (gate: float32 [rows, hidden]). */
 int roost_wide_rms_norm_gated(float* stream, const void* addend, const float* gate, const float* gate_bias, const float* w, void* out,
                               const int32_t* rows, int n_out, int hidden, float eps, int dtype, roost_stream_t stream_handle);
+/* A norm after a sublayer and the norm before the next in one pass: s = stream + addend / sqrt(mean(addend^2) + post_eps) * post_w, written
+ * back unless `rows` gathers; out = s / sqrt(mean(s^2) + eps) * w. The addend and out have `dtype`, everything else is float. */
+int roost_sandwich_norm(float* stream, const void* addend, const float* post_w, float post_eps, const float* w, void* out, const int32_t* rows,
+                        int n_out, int hidden, float eps, int dtype, roost_stream_t stream_handle);
 int roost_scale(float* x, int64_t n, float factor, roost_stream_t stream);   /* x *= factor */
 /* out = mean over the n (1 to 4) branches of xs[b] / sqrt(mean(xs[b]^2) + eps) * ws[b]. */
 int roost_normed_mean(const void* const* xs, const float* const* ws, int n, void* out, int tokens, int hidden, float eps, int dtype,
                       roost_stream_t stream);
+/* out = sum over the n (1 to 4) branches of ws[b] * xs[b], `count` numbers each (xs and ws are host arrays). */
+int roost_weighted_sum(const void* const* xs, const float* ws, int n, void* out, int64_t count, int dtype, roost_stream_t stream);
 /* out[t] = table[ids[t]] + pairs[row]: row = (previous id * mul_prev + id * mul_cur) mod buckets, `buckets` at position <= 0; the id
  * before a row's first token of the step is state[slots[row]]. */
 int roost_pair_embedding(const void* table, const void* pairs, const int32_t* ids, const int32_t* positions, const int32_t* token_row,
@@ -454,6 +462,35 @@ int roost_retention_scan(const float* qk, const void* v, int64_t ldv, float* out
                          const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, float* ws, int dtype,
                          roost_stream_t stream);
 
+/* The same where nothing is rotated, over the projection's rows u = [q heads | k heads | v heads | ...], ld apart: act 1 puts SiLU on q, k
+ * and v (0: nothing), the keys are multiplied by k_scale. */
+int roost_retention_scan_raw(const void* u, int64_t ld, int act, float k_scale, float* out, float* state, int64_t state_stride,
+                             const float* decay, const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim,
+                             int vdim, float* ws, int dtype, roost_stream_t stream);
+
+/* ---- the recurrence whose gates read only the current token (min_gru.cu) ---- */
+/* u rows [z | x | g], ld apart; z = sigmoid(z + z_bias), x = x + x_bias, c = x + 1/2 (x >= 0) or sigmoid(x); S <- (1 - z) S + z c; out
+ * (rows ld_out apart) = S silu(g) out_scale, rounded once. State slots [S: width | ...]. ws_state, ws_keep:
+ * float[roost_min_gru_scan_chunks(tokens, rows) * width] each, or both null; with them rows are cut into chunks of 16 tokens that run
+ * side by side (three launches). */
+int roost_min_gru_scan_chunks(int tokens, int rows);
+int roost_min_gru_scan(const void* u, int64_t ld, void* out, int64_t ld_out, const float* z_bias, const float* x_bias, float out_scale,
+                       float* state, int64_t state_stride, const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int width,
+                       float* ws_state, float* ws_keep, int dtype, roost_stream_t stream);
+
+/* ---- attention whose scores are mixed across the heads before the softmax (talking_attention.cu) ---- */
+/* q [tokens, heads, dim] (prepared queries; keys and values in the cache as roost_sink_attention_prepare leaves them). score'_h = scale *
+ * sum_g talk[h, g] (q_g . k_g), a softmax over the visible keys (the last `window`, the query's own included; 0: all), out[t, h] = its
+ * weighted values, times sigmoid(gate[t, h, :]) where gate is not null (rows ld_gate apart), times out_scale; out rows ld_out apart.
+ * splits > 1: a token's tiles of key_tile keys are dealt in ranges of tiles_per_split to `splits` blocks; part: float[tokens * heads *
+ * splits * (vdim + 2)]. key_tile: roost_talking_attention_key_tile(...), 0 where no tile fits the shared memory. */
+int roost_talking_attention_key_tile(int heads, int kv_heads, int dim, int vdim, int dtype);
+int roost_talking_attention(const void* q, void* out, int64_t ld_out, float* part, const void* k_base, const void* v_base, int entry,
+                            const void* gate, int64_t ld_gate, const float* talk, const int32_t* positions, const int32_t* token_row,
+                            const int32_t* kv_indptr, const int32_t* kv_indices, int tokens, int heads, int kv_heads, int dim, int vdim,
+                            int page_size, float scale, int window, float out_scale, int key_tile, int splits, int tiles_per_split, int dtype,
+                            roost_stream_t stream);
+
 /* ---- attention with sigmoid weights (sigmoid_attention.cu) ---- */
 /* Queries and keys divided by their root mean square times q_w / k_w (dim numbers each); queries times
  * 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) into q_out [tokens, heads, dim]; keys and values into the cache. */
@@ -491,6 +528,7 @@ int roost_carried_attention(const void* q, int64_t ld_q, void* out, const void* 
 /* ---- activations.cu ---- */
 /* y = a_pos z^2 + z / 2 (z > 0), a_neg (exp(z) - 1 - z) + z / 2 (z <= 0). */
 int roost_xielu(const void* x, void* out, int64_t n, float a_pos, float a_neg, int dtype, roost_stream_t stream);
+int roost_relu_squared(const void* x, void* out, int64_t n, int dtype, roost_stream_t stream);   /* y = max(z, 0)^2 */
 /* x[t, h, :] *= sigmoid(g[t, col + h]) in place; g's rows are ld_g apart. */
 int roost_head_gate_mul(void* x, const void* g, int64_t ld_g, int col, int tokens, int heads, int vdim, int dtype, roost_stream_t stream);
 

@@ -23,8 +23,6 @@ constexpr int kSgTile = 32;
 constexpr int kSgWarps = 8;
 constexpr int kSgMaxDim = 512;
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-
 template <typename T>
 __global__ void __launch_bounds__(128) sigmoid_prepare_kernel(const T* __restrict__ qkv, int64_t ld, T* __restrict__ q_out, T* k_base, T* v_base, int entry,
                                                              const float* __restrict__ q_w, const float* __restrict__ k_w,

@@ -4,7 +4,7 @@
 //   prepare:   per token, on a row [q heads | k heads | v heads] of the fused projection: every query and key head has its
 //              first rot_dims elements turned in interleaved pairs, (u, v) at (2i, 2i+1) -> (u cos a - v sin a, v cos a + u sin a)
 //              with a = position * inv_freq[i] formed in double and reduced to [-pi, pi] (with `halves` the pair is
-//              (i, i + rot_dims / 2) instead); then, with eps > 0, the head is
+//              (i, i + rot_dims / 2) instead; cosines and sines are both multiplied by `amplitude`); then, with eps > 0, the head is
 //              divided by sqrt(mean(x^2) + eps) (no weight). Queries are written back in place (or, with q_out, to a dense
 //              [tokens, heads, dim] tensor of their own, which the tensor-core attention kernels read), keys and values go to the
 //              token's cache slot (slot -1: nothing is written). The cache entry of (page, kv head, offset) starts at
@@ -12,8 +12,8 @@
 //              size, or one plane whose entries are [key | value] (v_base = k_base + dim, entry = dim + vdim).
 //   attention: one block per (token, key/value head, eight of its query heads, split); a warp a query head; key tiles of 32 at
 //              absolute positions staged in shared memory as float32; a lane a key for the scores, a lane a value column for
-//              the sums; running maximum and denominator a warp. The sink is a key of score 0 without a value: the running
-//              maximum starts at 0 and the denominator at 1. A token's tiles may be dealt to several blocks in ranges
+//              the sums; running maximum and denominator a warp. The sink is a key of score 0 (or of the head's stored score)
+//              without a value: the running maximum starts at that score and the denominator at 1. A token's tiles may be dealt to several blocks in ranges
 //              (split z of Z takes tiles [z n, (z + 1) n), n from the step's bound on lengths); the partial sums, maxima and
 //              denominators are then combined in split order by a second kernel. A padding token (position -1) is skipped.
 //              With a window a query at position p sees the keys p - window + 1 .. p: its tiles start at the tile of the first
@@ -31,7 +31,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) sink_prepare_kernel(T* qkv, int64_t ld, T* q_out, T* k_base, T* v_base, int entry, const double* __restrict__ inv_freq,
                                                           const int32_t* __restrict__ positions, const int32_t* __restrict__ slot_mapping,
                                                           int heads, int kv_heads, int dim, int vdim, int rot_dims, float eps, int page_size,
-                                                          int halves) {
+                                                          int halves, float amplitude) {
   extern __shared__ float sm[];      // rot_dims/2 cosines, rot_dims/2 sines
   const int half = rot_dims / 2;
   float* cs = sm;
@@ -43,6 +43,8 @@ __global__ void __launch_bounds__(128) sink_prepare_kernel(T* qkv, int64_t ld, T
     double ang = (double)pos * inv_freq[i];
     ang -= 6.283185307179586476925286766559 * rint(ang * 0.15915494309189533576888376337251);
     sincosf((float)ang, &sn[i], &cs[i]);
+    sn[i] *= amplitude;
+    cs[i] *= amplitude;
   }
   const int slot = slot_mapping[t];
   pdl_wait();
@@ -106,7 +108,8 @@ __global__ void __launch_bounds__(kSaWarps * 32) sink_attention_kernel(const T* 
                                                                      const int32_t* __restrict__ positions, const int32_t* __restrict__ token_row,
                                                                      const int32_t* __restrict__ kv_indptr, const int32_t* __restrict__ kv_indices,
                                                                      int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink,
-                                                                     int splits, int tiles_per_split, int window, float softcap) {
+                                                                     int splits, int tiles_per_split, int window, float softcap,
+                                                                     const float* __restrict__ sinks) {
   extern __shared__ float sm[];
   float* ks = sm;                                          // [tile][dim + 1]
   float* vs = ks + (size_t)kSaTile * (dim + 1);            // [tile][vdim]
@@ -132,8 +135,8 @@ __global__ void __launch_bounds__(kSaWarps * 32) sink_attention_kernel(const T* 
     for (int i = lane; i < dim; i += 32) qs[(size_t)warp * dim + i] = to_float(q[i]);
   }
   float m = -INFINITY, l = 0.f;
-  if (sink && z == 0) {
-    m = 0.f;
+  if (sink && z == 0 && active) {
+    m = sinks != nullptr ? sinks[h] : 0.f;
     l = 1.f;
   }
   float acc[kSaMaxDim / 32];
@@ -264,7 +267,8 @@ using namespace roost;
 
 extern "C" int roost_sink_attention_prepare(void* qkv, int64_t ld, void* q_out, void* k_base, void* v_base, int entry, const double* inv_freq,
                                             const int32_t* positions, const int32_t* slot_mapping, int tokens, int heads, int kv_heads, int dim,
-                                            int vdim, int rot_dims, float eps, int page_size, int halves, int dtype, roost_stream_t stream) {
+                                            int vdim, int rot_dims, float eps, int page_size, int halves, float amplitude, int dtype,
+                                            roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0, "sink_attention_prepare: sizes must be positive");
   ROOST_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim, "sink_attention_prepare: the rotated width must be even and at most dim");
   ROOST_REQUIRE(qkv && k_base && v_base && positions && slot_mapping && (rot_dims == 0 || inv_freq), "sink_attention_prepare: a pointer is null");
@@ -276,14 +280,14 @@ extern "C" int roost_sink_attention_prepare(void* qkv, int64_t ld, void* q_out, 
   // four warps a token: measured faster than a warp a head (sixteen warps: 30.7 against 19.6 us at 2,048 tokens of 16 + 4 heads of 64)
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(sink_prepare_kernel<T>, dim3(tokens), dim3(128), smem, (cudaStream_t)stream, (T*)qkv, ld, (T*)q_out, (T*)k_base,
                                                (T*)v_base, entry, inv_freq, positions, slot_mapping, heads, kv_heads, dim, vdim, rot_dims, eps,
-                                               page_size, halves));
+                                               page_size, halves, amplitude));
   return check_launch("sink_attention_prepare");
 }
 
 extern "C" int roost_sink_attention(const void* qkv, int64_t ld, void* out, float* part, const void* k_base, const void* v_base, int entry,
                                     const int32_t* positions, const int32_t* token_row, const int32_t* kv_indptr, const int32_t* kv_indices,
                                     int tokens, int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink, int splits,
-                                    int tiles_per_split, int window, float softcap, int dtype, roost_stream_t stream) {
+                                    int tiles_per_split, int window, float softcap, const float* sinks, int dtype, roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0, "sink_attention: sizes must be positive");
   ROOST_REQUIRE(heads % kv_heads == 0, "sink_attention: the query heads are no multiple of the key/value heads");
   ROOST_REQUIRE(window >= 0 && softcap >= 0.f, "sink_attention: the window and the scores' cap cannot be negative");
@@ -300,7 +304,7 @@ extern "C" int roost_sink_attention(const void* qkv, int64_t ld, void* out, floa
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(kernel, grid, dim3(kSaWarps * 32), smem, (cudaStream_t)stream, (const T*)qkv, ld, (T*)out, splits > 1 ? part : (float*)nullptr,
                   (const T*)k_base, (const T*)v_base, entry, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, page_size,
-                  scale, sink, splits, tiles_per_split, window, softcap);
+                  scale, sink, splits, tiles_per_split, window, softcap, sinks);
     if (splits > 1)
       launch_kernel(sink_merge_kernel<T>, dim3(tokens, heads), dim3(128), 0, (cudaStream_t)stream, (const float*)part, (T*)out, positions, heads,
                     vdim, splits);

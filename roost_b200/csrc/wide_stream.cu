@@ -92,6 +92,94 @@ __global__ void wide_rms_norm_kernel(float* stream, const T* __restrict__ addend
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = from_float<T>(row[i] * inv * w[i]);
 }
 
+// The norm after a sublayer and the norm before the next one in one pass over a 32-bit stream. One block per output row: the addend's
+// root mean square, s = stream + addend * inv * post_w (written back unless the rows are gathered), then s's root mean square and the
+// output, rounded once. Rows a block covers with eight numbers a thread stay in registers (VEC); others go through shared memory.
+template <typename T, bool VEC>
+__global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend, const float* __restrict__ post_w, float post_eps,
+                                     const float* __restrict__ w, T* __restrict__ out, const int32_t* __restrict__ rows, int hidden, float eps) {
+  extern __shared__ float row[];  // 32 floats of reduction scratch; without VEC `hidden` floats after them
+  float* scratch = row;
+  pdl_launch_dependents();
+  const int i_out = blockIdx.x;
+  const size_t r = rows ? (size_t)rows[i_out] : (size_t)i_out;
+  float* s_row = stream + r * hidden;
+  const T* a_row = addend + r * hidden;
+  T* o_row = out + (size_t)i_out * hidden;
+  if constexpr (VEC) {
+    const int i8 = threadIdx.x * 8;
+    const bool live = i8 < hidden;
+    float pw[8], nw[8], a[8], s[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) pw[j] = nw[j] = a[j] = s[j] = 0.f;
+    if (live) {      // weights do not depend on the kernel in front
+#pragma unroll
+      for (int j = 0; j < 8; j += 4) {
+        *reinterpret_cast<float4*>(pw + j) = *reinterpret_cast<const float4*>(post_w + i8 + j);
+        *reinterpret_cast<float4*>(nw + j) = *reinterpret_cast<const float4*>(w + i8 + j);
+      }
+    }
+    pdl_wait();
+    if (live) {
+      if constexpr (sizeof(T) == 2) {
+        Vec<T>::load(a_row + i8, a);
+      } else {
+        *reinterpret_cast<float4*>(a) = *reinterpret_cast<const float4*>(a_row + i8);
+        *reinterpret_cast<float4*>(a + 4) = *reinterpret_cast<const float4*>(a_row + i8 + 4);
+      }
+      *reinterpret_cast<float4*>(s) = *reinterpret_cast<const float4*>(s_row + i8);
+      *reinterpret_cast<float4*>(s + 4) = *reinterpret_cast<const float4*>(s_row + i8 + 4);
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(a[j], a[j], ss);
+    ss = block_sum(ss, scratch);
+    const float inv_a = 1.0f / sqrtf(ss / (float)hidden + post_eps);
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      s[j] = s[j] + a[j] * inv_a * pw[j];
+      ss = fmaf(s[j], s[j], ss);
+    }
+    ss = block_sum(ss, scratch);
+    if (!live) return;
+    if (!rows) {
+      *reinterpret_cast<float4*>(s_row + i8) = make_float4(s[0], s[1], s[2], s[3]);
+      *reinterpret_cast<float4*>(s_row + i8 + 4) = make_float4(s[4], s[5], s[6], s[7]);
+    }
+    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[j] = s[j] * inv * nw[j];
+    if constexpr (sizeof(T) == 2) {
+      Vec<T>::store(o_row + i8, s);
+    } else {
+      *reinterpret_cast<float4*>(o_row + i8) = make_float4(s[0], s[1], s[2], s[3]);
+      *reinterpret_cast<float4*>(o_row + i8 + 4) = make_float4(s[4], s[5], s[6], s[7]);
+    }
+  } else {
+    float* keep = row + 32;
+    pdl_wait();
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+      const float a = to_float(a_row[i]);
+      keep[i] = a;
+      ss = fmaf(a, a, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv_a = 1.0f / sqrtf(ss / (float)hidden + post_eps);
+    ss = 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {      // every thread meets the entries it wrote itself
+      const float s = s_row[i] + keep[i] * inv_a * post_w[i];
+      if (!rows) s_row[i] = s;
+      keep[i] = s;
+      ss = fmaf(s, s, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o_row[i] = from_float<T>(keep[i] * inv * w[i]);
+  }
+}
+
 // The mean of up to four branch outputs, each divided by its root mean square over the row and multiplied by its weight.
 struct NormedMeanArgs {
   const void* x[4];
@@ -160,6 +248,25 @@ __global__ void normed_mean_kernel(NormedMeanArgs a, int n, T* __restrict__ out,
     for (int b = 0; b < n; ++b) s = fmaf(to_float(reinterpret_cast<const T*>(a.x[b])[t * hidden + i]) * inv[b], a.w[b][i], s);
     out[t * hidden + i] = from_float<T>(s * share);
   }
+}
+
+// The sum of up to four branch outputs, each times a factor, formed in 32-bit and rounded once.
+struct WeightedSumArgs {
+  const void* x[4];
+  float w[4];
+};
+
+template <typename T>
+__global__ void weighted_sum_kernel(WeightedSumArgs a, int n, T* __restrict__ out, size_t count) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= count) return;
+  float s = 0.f;
+#pragma unroll
+  for (int b = 0; b < 4; ++b)
+    if (b < n) s = fmaf(a.w[b], to_float(reinterpret_cast<const T*>(a.x[b])[i]), s);
+  out[i] = from_float<T>(s);
 }
 
 // table[id] + pairs[row] as a 32-bit stream; row = (previous id * mul_prev + id * mul_cur) mod buckets, or `buckets` for a
@@ -308,6 +415,26 @@ extern "C" int roost_wide_rms_norm_gated(float* stream, const void* addend, cons
   return check_launch("wide_rms_norm_gated");
 }
 
+extern "C" int roost_sandwich_norm(float* stream, const void* addend, const float* post_w, float post_eps, const float* w, void* out,
+                                   const int32_t* rows, int n_out, int hidden, float eps, int dtype, roost_stream_t stream_handle) {
+  ROOST_REQUIRE(n_out >= 0 && hidden > 0, "sandwich_norm: rows and hidden must be positive");
+  ROOST_REQUIRE(eps > 0.f && post_eps > 0.f, "sandwich_norm: both eps must be positive");
+  ROOST_REQUIRE(stream && addend && post_w && w && out, "sandwich_norm: a pointer is null");
+  if (n_out == 0) return ROOST_OK;
+  const bool vec = hidden % 8 == 0 && hidden <= 8192 &&
+                   (((uintptr_t)stream | (uintptr_t)addend | (uintptr_t)post_w | (uintptr_t)w | (uintptr_t)out) % 16 == 0);
+  const size_t smem = vec ? 32 * sizeof(float) : ((size_t)hidden + 32) * sizeof(float);
+  if (smem > 200 * 1024) return fail(ROOST_ERR_UNSUPPORTED, "sandwich_norm: a row of more than 51168 elements does not fit in shared memory");
+  const int threads = vec ? (hidden / 8 + 31) / 32 * 32 : (hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128));
+  ROOST_DISPATCH_DTYPE(dtype, T, {
+    auto kernel = vec ? sandwich_norm_kernel<T, true> : sandwich_norm_kernel<T, false>;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    launch_kernel(kernel, dim3(n_out), dim3(threads), smem, (cudaStream_t)stream_handle, stream, (const T*)addend, post_w, post_eps, w, (T*)out, rows,
+                  hidden, eps);
+  });
+  return check_launch("sandwich_norm");
+}
+
 extern "C" int roost_scale(float* x, int64_t n, float factor, roost_stream_t stream) {
   ROOST_REQUIRE(n >= 0 && (n == 0 || x), "scale: a pointer is null");
   if (n == 0) return ROOST_OK;
@@ -331,6 +458,23 @@ extern "C" int roost_normed_mean(const void* const* xs, const float* const* ws, 
   const int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(normed_mean_kernel<T>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, a, n, (T*)out, hidden, eps));
   return check_launch("normed_mean");
+}
+
+extern "C" int roost_weighted_sum(const void* const* xs, const float* ws, int n, void* out, int64_t count, int dtype, roost_stream_t stream) {
+  ROOST_REQUIRE(n >= 1 && n <= 4, "weighted_sum: one to four branches");
+  ROOST_REQUIRE(count >= 0 && (count == 0 || (xs && ws && out)), "weighted_sum: a pointer is null");
+  if (count == 0) return ROOST_OK;
+  WeightedSumArgs a = {};
+  for (int b = 0; b < n; ++b) {
+    ROOST_REQUIRE(xs[b], "weighted_sum: a pointer is null");
+    a.x[b] = xs[b];
+    a.w[b] = ws[b];
+  }
+  const int64_t blocks = (count + 255) / 256;
+  if (blocks > 2147483647LL) return fail(ROOST_ERR_UNSUPPORTED, "weighted_sum: too many numbers for one launch");
+  ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(weighted_sum_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, a, n, (T*)out,
+                                               (size_t)count));
+  return check_launch("weighted_sum");
 }
 
 extern "C" int roost_pair_embedding(const void* table, const void* pairs, const int32_t* ids, const int32_t* positions, const int32_t* token_row,

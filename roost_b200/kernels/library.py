@@ -14,7 +14,7 @@ import torch
 
 from . import build
 
-ABI_VERSION = 15
+ABI_VERSION = 16
 F32, BF16 = 0, 1
 GATE_FUNCTIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}   # the codes of csrc/roost_kernels.h
 
@@ -56,6 +56,16 @@ def _need(t: torch.Tensor, name: str, dtype=None):
         raise KernelError(f"{name} has dtype {t.dtype}; expected {dtype}")
 
 
+def _need_rows(t: torch.Tensor, name: str, dtype=None):
+    """A matrix whose rows are dense and may lie apart (a range of the columns of a wider one)."""
+    if not t.is_cuda:
+        raise KernelError(f"{name} is not on a CUDA device")
+    if t.dim() != 2 or (t.shape[1] > 1 and t.stride(1) != 1) or (t.shape[0] > 1 and t.stride(0) < t.shape[1]):
+        raise KernelError(f"{name} is not a matrix with dense rows")
+    if dtype is not None and t.dtype != dtype:
+        raise KernelError(f"{name} has dtype {t.dtype}; expected {dtype}")
+
+
 _SIGNATURES = {
     "roost_status_snapshot": [c_void_p, c_int, c_void_p],
     "roost_embedding": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -74,14 +84,14 @@ _SIGNATURES = {
     "roost_attention_set_prefill_tc": [c_int],
     "roost_attention_prefill_tile_rows_mma": [c_int, c_int, ctypes.c_longlong],
     "roost_attention_prefill": [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p],
+                                c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p, c_void_p],
     "roost_attention_prefill_capped": [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                       c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_float, c_void_p],
+                                       c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_float, c_void_p, c_void_p],
     "roost_attention_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int,
-                               c_void_p],
+                               c_void_p, c_void_p],
     "roost_attention_decode_cluster": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                       c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p],
+                                       c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p, c_void_p],
     "roost_attention_decode_cluster_supported": [c_int, c_int, ctypes.c_longlong, c_int, c_void_p, c_void_p],
     "roost_sample_penalise": [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_void_p],
@@ -141,9 +151,9 @@ _SIGNATURES = {
                           c_int, c_void_p],
     "roost_gated_act_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
     "roost_sink_attention_prepare": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                     c_int, c_float, c_int, c_int, c_int, c_void_p],
+                                     c_int, c_float, c_int, c_int, c_float, c_int, c_void_p],
     "roost_sink_attention": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+                             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "roost_wide_rms_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "roost_normed_mean": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "roost_pair_embedding": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -173,6 +183,18 @@ _SIGNATURES = {
     "roost_carried_attention_supported": [c_int, c_int],
     "roost_carried_attention": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                 c_void_p],
+    "roost_retention_scan_raw": [c_void_p, c_int64, c_int, c_float, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                                 c_int, c_void_p, c_int, c_void_p],
+    "roost_min_gru_scan_chunks": [c_int, c_int],
+    "roost_min_gru_scan": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
+                           c_void_p, c_void_p, c_int, c_void_p],
+    "roost_talking_attention_key_tile": [c_int, c_int, c_int, c_int, c_int],
+    "roost_talking_attention": [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_int, c_int, c_int,
+                                c_void_p],
+    "roost_relu_squared": [c_void_p, c_void_p, c_int64, c_int, c_void_p],
+    "roost_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
+    "roost_weighted_sum": [c_void_p, c_void_p, c_int, c_void_p, c_int64, c_int, c_void_p],
     "roost_xielu": [c_void_p, c_void_p, c_int64, c_float, c_float, c_int, c_void_p],
     "roost_head_gate_mul": [c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "roost_wide_rms_norm_gated": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
@@ -411,9 +433,11 @@ class KernelLibrary:
     ATTENTION_WIDE_WEIGHTS = 1 << 29
 
     def attention_mma(self, q, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, plan, scale: float,
-                      window: int | None, sink: bool = False, wide_weights: bool = False, softcap: float = 0.0) -> torch.Tensor:
+                      window: int | None, sink: bool = False, wide_weights: bool = False, softcap: float = 0.0,
+                      sinks: torch.Tensor | None = None) -> torch.Tensor:
         """Tensor-core attention (bfloat16). ``plan``: an ``AttentionPlan`` whose work lists are on the device. ``sink``: one is
-        added to the softmax's denominator (a key of score 0 that has no value). ``wide_weights``: the softmax weights enter P V as two
+        added to the softmax's denominator (a key of score 0 that has no value), or exp(sinks[h]) of head h with ``sinks`` (float32, one a
+        query head). ``wide_weights``: the softmax weights enter P V as two
         bfloat16 operands (16 bits of the 32-bit weights); the plan's prefill items must then come from
         ``attention_prefill_tile_rows(..., tensor_memory=False)``. ``softcap`` c > 0: a scaled score s becomes c tanh(s / c); the
         prompt kernels on mma.sync serve it (items from ``tensor_memory=False``), the decode kernels do not: the plan must hold no
@@ -425,20 +449,24 @@ class KernelLibrary:
             raise KernelError("attention_mma: head_dim of q and of the pool differ")
         out = torch.empty((T, nq * d), dtype=q.dtype, device=q.device)
         w = (int(window) if window else 0) | (self.ATTENTION_SINK if sink else 0) | (self.ATTENTION_WIDE_WEIGHTS if wide_weights else 0)
+        if sinks is not None:
+            _need(sinks, "sinks", torch.float32)
+            if not sink or sinks.numel() != nq:
+                raise KernelError("attention_mma: stored sinks come with ``sink`` and are one number a query head")
         if softcap and plan.decode_items:
             raise KernelError("attention_mma: the decode kernels know no cap on the scores")
         if plan.prefill_items and softcap:
             self._call("roost_attention_prefill_capped", _ptr(q), T, _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.prefill_work), plan.prefill_items, plan.prefill_tile_rows, nq, nkv, d, page,
-                       k_pool.shape[0], scale, w, float(softcap), _stream())
+                       k_pool.shape[0], scale, w, float(softcap), _ptr(sinks), _stream())
         elif plan.prefill_items:
             self._call("roost_attention_prefill", _ptr(q), T, _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.prefill_work), plan.prefill_items, plan.prefill_tile_rows, nq, nkv, d, page,
-                       k_pool.shape[0], scale, w, _stream())
+                       k_pool.shape[0], scale, w, _ptr(sinks), _stream())
         if plan.decode_items and plan.cluster_chunks:
             self._call("roost_attention_decode_cluster", _ptr(q), _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.decode_work), plan.decode_items, plan.cluster_chunks, nq, nkv, d, page,
-                       k_pool.shape[0], scale, w, _stream())
+                       k_pool.shape[0], scale, w, _ptr(sinks), _stream())
         elif plan.decode_items:
             part_o = part_ml = None
             if plan.slots:
@@ -446,7 +474,7 @@ class KernelLibrary:
                 part_ml = torch.empty((plan.slots * nkv * 16 * 2,), dtype=torch.float32, device=q.device)
             self._call("roost_attention_decode", _ptr(q), _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.decode_work), plan.decode_items, _ptr(plan.merge_work),
-                       plan.merge_items, plan.merge_rows, _ptr(part_o), _ptr(part_ml), nq, nkv, d, page, k_pool.shape[0], scale, w, _stream(),
+                       plan.merge_items, plan.merge_rows, _ptr(part_o), _ptr(part_ml), nq, nkv, d, page, k_pool.shape[0], scale, w, _ptr(sinks), _stream(),
                        launches=2 if plan.merge_items else 1)
         return out
 
@@ -917,24 +945,25 @@ class KernelLibrary:
         return k_pool.data_ptr(), v_pool.data_ptr(), dim
 
     def sink_attention_prepare(self, qkv, k_pool, v_pool, inv_freq, rotary_dim, positions, slot_mapping, heads, kv_heads, dim, vdim, eps,
-                               page_size, q_out: torch.Tensor | None = None, halves: bool = False) -> None:
+                               page_size, q_out: torch.Tensor | None = None, halves: bool = False, amplitude: float = 1.0) -> None:
         """``q_out`` [tokens, heads, dim]: where the prepared queries go instead of back into ``qkv``. ``halves``: element i of the
-        rotated part is paired with element i + rotary_dim / 2 instead of its neighbour."""
+        rotated part is paired with element i + rotary_dim / 2 instead of its neighbour. ``amplitude`` multiplies cosines and sines. ``qkv``
+        may be a range of the columns of wider rows."""
         if q_out is not None:
             _need(q_out, "q_out", qkv.dtype)
             if tuple(q_out.shape) != (qkv.shape[0], heads, dim):
                 raise KernelError("sink_attention_prepare: q_out is not [tokens, heads, dim]")
-        _need(qkv, "qkv"); _need(k_pool, "k_pool", qkv.dtype); _need(positions, "positions", torch.int32); _need(slot_mapping, "slot_mapping", torch.int32)
+        _need_rows(qkv, "qkv"); _need(k_pool, "k_pool", qkv.dtype); _need(positions, "positions", torch.int32); _need(slot_mapping, "slot_mapping", torch.int32)
         if v_pool is not None:
             _need(v_pool, "v_pool", qkv.dtype)
         if rotary_dim:
             _need(inv_freq, "inv_freq", torch.float64)
-        if qkv.shape[1] != (heads + kv_heads) * dim + kv_heads * vdim or k_pool.shape[1] != kv_heads or k_pool.shape[2] != page_size:
+        if qkv.shape[1] < (heads + kv_heads) * dim + kv_heads * vdim or k_pool.shape[1] != kv_heads or k_pool.shape[2] != page_size:
             raise KernelError("sink_attention_prepare: qkv or the pool do not fit the sizes")
         kb, vb, entry = self._sink_cache(k_pool, v_pool, dim, vdim)
         self._call("roost_sink_attention_prepare", _ptr(qkv), qkv.stride(0), _ptr(q_out), kb, vb, entry, _ptr(inv_freq) if rotary_dim else None, _ptr(positions),
                    _ptr(slot_mapping), qkv.shape[0], heads, kv_heads, dim, vdim, rotary_dim, float(eps) if eps else 0.0, page_size,
-                   1 if halves else 0, dtype_code(qkv.dtype), _stream())
+                   1 if halves else 0, float(amplitude), dtype_code(qkv.dtype), _stream())
 
     def sink_splits_for(self, tokens: int, gy: int, kv_cap: int) -> tuple[int, int]:
         """(blocks a token's key tiles are dealt to, tiles a block): 1 when the step's blocks fill the device by themselves,
@@ -948,12 +977,17 @@ class KernelLibrary:
         return -(-tiles // per), per
 
     def sink_attention(self, qkv, k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, scale, sink,
-                       kv_cap: int = 0, window: int | None = None, softcap: float = 0.0) -> torch.Tensor:
+                       kv_cap: int = 0, window: int | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None) -> torch.Tensor:
         """Attention of the step's (prepared) queries over the paged cache in 32-bit arithmetic: out [T, heads * vdim]. ``window``:
-        the keys a query sees, its own included (None: all); ``softcap`` c > 0: a scaled score s becomes c tanh(s / c)."""
+        the keys a query sees, its own included (None: all); ``softcap`` c > 0: a scaled score s becomes c tanh(s / c); ``sinks`` (float32, one
+        a query head): exp(sinks[h]) is the sink's term in the denominator instead of one."""
         _need(qkv, "qkv"); _need(k_pool, "k_pool", qkv.dtype)
         for n, t in (("positions", positions), ("token_row", token_row), ("kv_indptr", kv_indptr), ("kv_indices", kv_indices)):
             _need(t, n, torch.int32)
+        if sinks is not None:
+            _need(sinks, "sinks", torch.float32)
+            if not sink or sinks.numel() != heads:
+                raise KernelError("sink_attention: stored sinks come with ``sink`` and are one number a query head")
         T = qkv.shape[0]
         kb, vb, entry = self._sink_cache(k_pool, v_pool, dim, vdim)
         out = torch.empty((T, heads * vdim), dtype=qkv.dtype, device=qkv.device)
@@ -964,7 +998,7 @@ class KernelLibrary:
         part = torch.empty((T * heads * splits * (vdim + 2),), dtype=torch.float32, device=qkv.device) if splits > 1 else None
         self._call("roost_sink_attention", _ptr(qkv), qkv.stride(0), _ptr(out), _ptr(part), kb, vb, entry, _ptr(positions), _ptr(token_row),
                    _ptr(kv_indptr), _ptr(kv_indices), T, heads, kv_heads, dim, vdim, k_pool.shape[2], float(scale), 1 if sink else 0, splits, per,
-                   int(window or 0), float(softcap or 0.0), dtype_code(qkv.dtype), _stream(), launches=2 if splits > 1 else 1)
+                   int(window or 0), float(softcap or 0.0), _ptr(sinks), dtype_code(qkv.dtype), _stream(), launches=2 if splits > 1 else 1)
         return out
 
     # ------------------------------------------------------------------ a 32-bit stream with root-mean-square norms
@@ -992,6 +1026,37 @@ class KernelLibrary:
         out = torch.empty((n, H), dtype=out_dtype, device=stream.device)
         self._call("roost_wide_rms_norm", _ptr(stream), _ptr(addend), _ptr(extra), _ptr(w), _ptr(out), _ptr(rows), n, H, eps, dtype_code(out_dtype),
                    _stream())
+        return out
+
+    def sandwich_norm(self, stream: torch.Tensor, addend: torch.Tensor, post_w: torch.Tensor, post_eps: float, w: torch.Tensor, eps: float,
+                      rows: torch.Tensor | None = None) -> torch.Tensor:
+        """The float32 ``stream`` plus the root-mean-square norm of ``addend`` (activation dtype) under ``post_w``, written back unless
+        ``rows`` gathers; returns the norm of the sum under ``w`` in the addend's dtype."""
+        _need(stream, "stream", torch.float32); _need(addend, "addend"); _need(post_w, "post_w", torch.float32); _need(w, "w", torch.float32)
+        H = stream.shape[-1]
+        if addend.shape != stream.shape or post_w.numel() != H or w.numel() != H:
+            raise KernelError("sandwich_norm: the stream, the addend and the weights differ in width")
+        if rows is not None:
+            _need(rows, "rows", torch.int32)
+        n = stream.numel() // H if rows is None else rows.numel()
+        out = torch.empty((n, H), dtype=addend.dtype, device=stream.device)
+        self._call("roost_sandwich_norm", _ptr(stream), _ptr(addend), _ptr(post_w), float(post_eps), _ptr(w), _ptr(out), _ptr(rows), n, H, float(eps),
+                   dtype_code(addend.dtype), _stream())
+        return out
+
+    def weighted_sum(self, xs: list, ws: list) -> torch.Tensor:
+        """sum over the branches of ws[b] * xs[b], formed in 32-bit and rounded once."""
+        n = len(xs)
+        if not 1 <= n <= 4 or len(ws) != n:
+            raise KernelError("weighted_sum: one to four branches with a factor each")
+        for x in xs:
+            _need(x, "x", xs[0].dtype)
+            if x.shape != xs[0].shape:
+                raise KernelError("weighted_sum: the branches differ in shape")
+        out = torch.empty_like(xs[0])
+        xp = (c_void_p * n)(*[x.data_ptr() for x in xs])
+        wp = (c_float * n)(*[float(w) for w in ws])
+        self._call("roost_weighted_sum", xp, wp, n, _ptr(out), out.numel(), dtype_code(out.dtype), _stream())
         return out
 
     def normed_mean(self, xs: list, ws: list, eps: float) -> torch.Tensor:
@@ -1131,6 +1196,85 @@ class KernelLibrary:
                    launches=3 if ws is not None else 1)
         return out
 
+    def retention_scan_raw(self, u, state, decay, q_indptr, slots, heads: int, dim: int, vdim: int, activation: str = "none", k_scale: float = 1.0,
+                           chunked: bool | None = None) -> torch.Tensor:
+        """The same where nothing is rotated, over the projection's rows ``u`` = [q heads | k heads | v heads | ...]: ``activation`` "silu"
+        puts SiLU on q, k and v, the keys are multiplied by ``k_scale``."""
+        if activation not in ("none", "silu"):
+            raise KernelError(f"retention_scan_raw: activation '{activation}' is neither none nor silu")
+        _need_rows(u, "u"); _need(state, "state", torch.float32); _need(decay, "decay", torch.float32)
+        _need(q_indptr, "q_indptr", torch.int32); _need(slots, "slots", torch.int32)
+        T = u.shape[0]
+        if u.shape[1] < heads * (2 * dim + vdim) or decay.numel() != heads:
+            raise KernelError("retention_scan_raw: the rows or the decays do not fit the sizes")
+        out = torch.empty((T, heads * vdim), dtype=torch.float32, device=u.device)
+        ws = None
+        if (T >= self.SCAN_CHUNKED_MIN_TOKENS) if chunked is None else chunked:
+            chunks = self._lib.roost_retention_scan_chunks(T, slots.numel())
+            ws = torch.empty((chunks * heads * dim * vdim,), dtype=torch.float32, device=u.device)
+        self._call("roost_retention_scan_raw", _ptr(u), u.stride(0), 1 if activation == "silu" else 0, float(k_scale), _ptr(out), _ptr(state),
+                   state.stride(0), _ptr(decay), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, _ptr(ws), dtype_code(u.dtype), _stream(),
+                   launches=3 if ws is not None else 1)
+        return out
+
+    # ------------------------------------------------------------------ the recurrence whose gates read only the current token
+    def min_gru_scan(self, u, out, z_bias, x_bias, out_scale: float, state, q_indptr, slots, width: int, chunked: bool | None = None) -> None:
+        """S <- (1 - z) S + z c a channel from rows [z | x | g] of ``u``; ``out`` (rows may lie apart) = S silu(g) ``out_scale``: see
+        csrc/min_gru.cu. ``chunked`` None: steps of ``SCAN_CHUNKED_MIN_TOKENS`` tokens or more cut their rows into chunks."""
+        _need_rows(u, "u"); _need_rows(out, "out", u.dtype); _need(state, "state", torch.float32)
+        _need(z_bias, "z_bias", torch.float32); _need(x_bias, "x_bias", torch.float32)
+        _need(q_indptr, "q_indptr", torch.int32); _need(slots, "slots", torch.int32)
+        T = u.shape[0]
+        if u.shape[1] < 3 * width or tuple(out.shape) != (T, width) or z_bias.numel() != width or x_bias.numel() != width:
+            raise KernelError("min_gru_scan: the rows or biases do not fit the sizes")
+        ws_state = ws_keep = None
+        if (T >= self.SCAN_CHUNKED_MIN_TOKENS) if chunked is None else chunked:
+            chunks = self._lib.roost_min_gru_scan_chunks(T, slots.numel())
+            ws_state = torch.empty((chunks * width,), dtype=torch.float32, device=u.device)
+            ws_keep = torch.empty((chunks * width,), dtype=torch.float32, device=u.device)
+        self._call("roost_min_gru_scan", _ptr(u), u.stride(0), _ptr(out), out.stride(0), _ptr(z_bias), _ptr(x_bias), float(out_scale), _ptr(state),
+                   state.stride(0), _ptr(q_indptr), _ptr(slots), slots.numel(), T, width, _ptr(ws_state), _ptr(ws_keep), dtype_code(u.dtype), _stream(),
+                   launches=3 if ws_state is not None else 1)
+
+    # ------------------------------------------------------------------ attention whose scores are mixed across the heads
+    def talking_key_tile(self, heads: int, kv_heads: int, dim: int, vdim: int, dtype: torch.dtype) -> int:
+        """Keys a tile of the 32-bit form of ``talking_attention`` holds at these sizes; 0: the heads do not fit the shared memory."""
+        return int(self._lib.roost_talking_attention_key_tile(heads, kv_heads, dim, vdim, dtype_code(dtype)))
+
+    def talking_splits_for(self, tokens: int, key_tile: int, span: int) -> tuple[int, int]:
+        """(blocks a token's key tiles are dealt to, tiles a block) for a step whose tokens see at most ``span`` keys: as many as give two
+        blocks an SM, up to 32 and to the tiles of the span; the last block takes what a longer row has left."""
+        if not self._decode_ctas:
+            self._decode_ctas = 2 * torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
+        tiles = -(-max(span, 1) // key_tile)
+        splits = max(1, min(self._decode_ctas // max(tokens, 1), tiles, 32))
+        per = -(-tiles // splits)
+        return -(-tiles // per), per
+
+    def talking_attention(self, q, out, k_pool, v_pool, gate, talk, positions, token_row, kv_indptr, kv_indices, kv_heads: int, vdim: int, scale: float,
+                          window: int | None = None, out_scale: float = 1.0, kv_cap: int = 0) -> None:
+        """Attention of the prepared queries q [T, heads, dim] whose scores are mixed across the heads by ``talk`` [heads, heads] before the
+        softmax, times sigmoid(``gate``) (rows may lie apart; None: no gate) and ``out_scale``, into ``out`` [T, heads * vdim]."""
+        _need(q, "q"); _need_rows(out, "out", q.dtype); _need(k_pool, "k_pool", q.dtype); _need(talk, "talk", torch.float32)
+        for n, t in (("positions", positions), ("token_row", token_row), ("kv_indptr", kv_indptr), ("kv_indices", kv_indices)):
+            _need(t, n, torch.int32)
+        T, heads, dim = q.shape
+        if gate is not None:
+            _need_rows(gate, "gate", q.dtype)
+            if tuple(gate.shape) != (T, heads * vdim):
+                raise KernelError("talking_attention: the gate's rows do not fit the sizes")
+        if tuple(out.shape) != (T, heads * vdim) or tuple(talk.shape) != (heads, heads):
+            raise KernelError("talking_attention: out or the mixing matrix do not fit the sizes")
+        kb, vb, entry = self._sink_cache(k_pool, v_pool, dim, vdim)
+        kt = self.talking_key_tile(heads, kv_heads, dim, vdim, q.dtype)
+        # a window's keys span at most window + key_tile - 1 positions' worth of tiles, whatever the requests' lengths are
+        span = min(kv_cap, window + 2 * kt - 2) if (window and kv_cap) else kv_cap
+        splits, per = self.talking_splits_for(T, kt, span) if (span and kt) else (1, 1 << 24)
+        part = torch.empty((T * heads * splits * (vdim + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
+        self._call("roost_talking_attention", _ptr(q), _ptr(out), out.stride(0), _ptr(part), kb, vb, entry, _ptr(gate), gate.stride(0) if gate is not None else 0,
+                   _ptr(talk), _ptr(positions), _ptr(token_row), _ptr(kv_indptr), _ptr(kv_indices), T, heads, kv_heads, dim, vdim, k_pool.shape[2],
+                   float(scale), int(window or 0), float(out_scale), kt, splits, per, dtype_code(q.dtype), _stream(), launches=2 if splits > 1 else 1)
+
     # ------------------------------------------------------------------ attention with sigmoid weights
     def sigmoid_attention_prepare(self, qkv, k_pool, v_pool, q_w, k_w, positions, slot_mapping, heads, kv_heads, dim, vdim, eps, temp_coef,
                                   temp_every, page_size) -> torch.Tensor:
@@ -1198,6 +1342,12 @@ class KernelLibrary:
         return out
 
     # ------------------------------------------------------------------ activations, gates, scaled sums
+    def relu_squared(self, x: torch.Tensor) -> torch.Tensor:
+        _need(x, "x")
+        out = torch.empty_like(x)
+        self._call("roost_relu_squared", _ptr(x), _ptr(out), x.numel(), dtype_code(x.dtype), _stream())
+        return out
+
     def xielu(self, x: torch.Tensor, a_pos: float, a_neg: float) -> torch.Tensor:
         """a_pos z^2 + z / 2 for z > 0, a_neg (exp(z) - 1 - z) + z / 2 for z <= 0."""
         _need(x, "x")

@@ -17,6 +17,7 @@ from ..config.spec import AttentionSpec
 from .attention_work import AttentionPlan, attention_caps, attention_work
 from .base import NORMS, POSITIONS, CacheNeed, Mixer, ParamDecl, Runtime, register_mixer
 from .linear import Linear
+from .positions import require_plain_amplitude
 
 SHORT_ROW_TOKENS = 16   # rows of at most this many tokens may go to the split decode kernel
 
@@ -50,6 +51,7 @@ class PagedAttention(Mixer):
             self.q_norm = NORMS.build(s.qk_norm, runtime)
             self.k_norm = NORMS.build(s.qk_norm, runtime)
         self.position = POSITIONS.build(s.position, runtime) if s.position is not None else None
+        require_plain_amplitude(self.position, "paged_attention")
 
     @classmethod
     def parameters(cls, spec: AttentionSpec):

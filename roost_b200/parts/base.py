@@ -109,6 +109,27 @@ class Mixer(Part):
         branch (a ``CacheNeed`` or None); its call then gets a tuple of cache views in the same order."""
         return None
 
+    # ---- splitting (optional). A mixer that is one product with its input, a middle part and one output projection may let a mixer of
+    # several side by side make the branches' input products in one and their output projections in one. It then sets ``splits``,
+    # loads through the three methods below, and its middle part reads its columns of the wide product ``u`` (rows may lie apart) and
+    # writes ``scale`` times its result into its columns ``out`` of what the wide output projection reads.
+    splits = False
+
+    def input_weight(self, params: dict) -> tuple:
+        """(weight [columns of u, hidden], bias [columns of u] or None)."""
+        raise NotImplementedError
+
+    def output_weight(self, params: dict) -> tuple:
+        """(weight [hidden, columns of out], bias [hidden] or None)."""
+        raise NotImplementedError
+
+    def load_middle(self, params: dict) -> None:
+        """Takes the parameters that belong to neither product."""
+        raise NotImplementedError
+
+    def middle(self, u: torch.Tensor, out: torch.Tensor, scale: float, batch, cache) -> None:
+        raise NotImplementedError
+
     # ---- per-step work lists (optional). A mixer whose kernels want lists derived on the host from the step's rows
     # (how the rows are divided among kernels and CTAs) asks the batch for them in its call: ``batch.step_work(self,
     # key)``. The batch calls back here. Neither the batch nor the executor knows what the lists hold: a captured step

@@ -173,6 +173,69 @@ class PreNormGatedBlock(Block):
         return norm.add_norm(h, residual.stream, rows=rows, gate=residual.gate)[0]
 
 
+class NormedStream:
+    """The 32-bit residual between two sublayers of a sandwich arrangement, and the norm that the branch output travelling beside it
+    still has to pass when it is added."""
+    __slots__ = ("stream", "post")
+
+    def __init__(self, stream, post):
+        self.stream, self.post = stream, post
+
+
+class SandwichWideBlock(Block):
+    """x <- x + out_norm1(mixer(norm1(x))); x <- x + out_norm2(ff(norm2(x))) over a residual kept and summed in 32-bit. A sublayer's output
+    passes its own norm in the kernel that adds it to the residual and norms the sum for the sublayer after it. The block hands on its last
+    branch output and the residual with the norm still to be applied; ``close`` does the last sum and the final norm of the wanted rows."""
+
+    def __init__(self, spec: BlockSpec, runtime: Runtime):
+        if spec.mixer_out_norm is None or (spec.feed_forward is not None and (spec.post_mixer_norm is None or spec.feed_forward_out_norm is None)):
+            raise ValueError("sandwich_wide: every sublayer needs the norm before it and the norm after it")
+        self.spec = spec
+        self.rt = runtime
+        self.input_norm = NORMS.build(spec.input_norm, runtime)
+        self.mixer = MIXERS.build(spec.mixer, runtime)
+        self.mixer_out_norm = NORMS.build(spec.mixer_out_norm, runtime)
+        self.feed_forward = self.post_mixer_norm = self.feed_forward_out_norm = None
+        if spec.feed_forward is not None:
+            self.post_mixer_norm = NORMS.build(spec.post_mixer_norm, runtime)
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, runtime)
+            self.feed_forward_out_norm = NORMS.build(spec.feed_forward_out_norm, runtime)
+
+    def sub_parts(self):
+        parts = {"input_norm": self.input_norm, "mixer": self.mixer, "mixer_out_norm": self.mixer_out_norm}
+        if self.feed_forward is not None:
+            parts.update({"post_mixer_norm": self.post_mixer_norm, "feed_forward": self.feed_forward,
+                          "feed_forward_out_norm": self.feed_forward_out_norm})
+        return parts
+
+    @classmethod
+    def sub_specs(cls, spec: BlockSpec):
+        subs = {"input_norm": (NORMS, spec.input_norm), "mixer": (MIXERS, spec.mixer), "mixer_out_norm": (NORMS, spec.mixer_out_norm)}
+        if spec.feed_forward is not None:
+            subs.update({"post_mixer_norm": (NORMS, spec.post_mixer_norm), "feed_forward": (FEED_FORWARDS, spec.feed_forward),
+                         "feed_forward_out_norm": (NORMS, spec.feed_forward_out_norm)})
+        return subs
+
+    def __call__(self, h, residual, batch, cache, write_cache: bool = True):
+        if residual is None:
+            if h.dtype != torch.float32:
+                raise ValueError("sandwich_wide: the embedding must hand over a float32 stream")
+            stream = h
+            x = self.input_norm(h)
+        else:
+            stream = residual.stream
+            x, _ = self.input_norm.add_norm(h, stream, post=residual.post)
+        a, post = self.mixer(x, batch, cache, write_cache), self.mixer_out_norm
+        if self.feed_forward is not None:
+            y, _ = self.post_mixer_norm.add_norm(a, stream, post=post)
+            a, post = self.feed_forward(y, batch), self.feed_forward_out_norm
+        return a, NormedStream(stream, post)
+
+    def close(self, h, residual, norm, rows):
+        """The model's end: the last normed sum of the wanted rows and ``norm`` of it."""
+        return norm.add_norm(h, residual.stream, rows=rows, post=residual.post)[0]
+
+
 class StreamState:
     """The residual streams between two sublayers: the 32-bit tensor [tokens, streams, width] and the connection whose
     write-back of the branch output that travels beside it is still to be applied."""
@@ -245,6 +308,7 @@ class PreNormStreamsBlock(Block):
         return self._read(h, residual, None, norm, rows=rows)[0]
 
 
+register_block("sandwich_wide", SandwichWideBlock)
 register_block("pre_norm_streams", PreNormStreamsBlock)
 register_block("pre_norm_gated", PreNormGatedBlock)
 register_block("pre_norm", PreNormBlock)

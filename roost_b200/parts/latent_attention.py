@@ -25,6 +25,7 @@ import torch
 from ..config.spec import LatentAttentionSpec
 from .base import POSITIONS, CacheNeed, Mixer, ParamDecl, Runtime, register_mixer
 from .linear import Linear, batched_linear
+from .positions import require_plain_amplitude
 
 
 class LatentAttention(Mixer):
@@ -52,6 +53,7 @@ class LatentAttention(Mixer):
         self.down = Linear(runtime, self.entry, s.hidden) if s.own_latent else None
         self.out = Linear(runtime, s.hidden, s.num_heads * s.v_dim)
         self.position = POSITIONS.build(s.position, runtime) if s.rope_dim else None
+        require_plain_amplitude(self.position, "latent_attention")
         self.head_gate = Linear(runtime, s.num_heads, s.hidden) if s.head_gate else None
         # Prompt portions of a run without a rotated part and without a window may leave the latent space: the rows' cached latents
         # are carried out to keys and values a head by two products, and the attention runs over those, a quarter of the products

@@ -88,9 +88,9 @@ class GatedMlp(FeedForward):
 class DenseMlp(FeedForward):
     """down(act(x Wu^T)) without a gate. ``xielu``: two stored numbers (p, q) give a_pos = softplus(p) and a_neg = 1/2 + softplus(q),
     formed once at load in double; act(z) = a_pos z^2 + z / 2 for z > 0 and a_neg (exp(z) - 1 - z) + z / 2 for z <= 0, on the 32-bit
-    value of the up projection's output, rounded once."""
+    value of the up projection's output, rounded once. ``relu_squared``: max(z, 0)^2 likewise, nothing stored."""
 
-    ACTIVATIONS = ("xielu",)
+    ACTIVATIONS = ("xielu", "relu_squared")
 
     def __init__(self, spec: DenseMlpSpec, runtime: Runtime):
         if spec.hidden <= 0 or spec.intermediate <= 0:
@@ -105,16 +105,23 @@ class DenseMlp(FeedForward):
     @classmethod
     def parameters(cls, spec: DenseMlpSpec):
         I, H = spec.intermediate, spec.hidden
-        return {"up": ParamDecl(shape=(I, H)), "down": ParamDecl(shape=(H, I)), "act": ParamDecl(shape=(2,), role="vector", init=("normal", 0.0, 0.5))}
+        decls = {"up": ParamDecl(shape=(I, H)), "down": ParamDecl(shape=(H, I))}
+        if spec.activation == "xielu":
+            decls["act"] = ParamDecl(shape=(2,), role="vector", init=("normal", 0.0, 0.5))
+        return decls
 
     def load(self, params):
         self.up.load(params["up"])
         self.down.load(params["down"])
+        if self.spec.activation != "xielu":
+            return
         p, q = (float(v) for v in params["act"].double().cpu())
         softplus = lambda z: max(z, 0.0) + math.log1p(math.exp(-abs(z)))
         self.a_pos, self.a_neg = softplus(p), 0.5 + softplus(q)
 
     def __call__(self, x, batch=None):
+        if self.spec.activation == "relu_squared":
+            return self.down(self.rt.kernels.relu_squared(self.up(x)))
         return self.down(self.rt.kernels.xielu(self.up(x), self.a_pos, self.a_neg))
 
 

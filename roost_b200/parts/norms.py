@@ -79,7 +79,9 @@ class WideRmsNorm(Norm):
 
     @classmethod
     def parameters(cls, spec: NormSpec):
-        return {"weight": ParamDecl(shape=(spec.size,), role="vector")}
+        # a weight stored around zero is drawn around zero
+        init = ("normal", 1.0 - spec.weight_offset, 0.05) if spec.weight_offset else None
+        return {"weight": ParamDecl(shape=(spec.size,), role="vector", init=init)}
 
     def load(self, params):
         self.weight = (params["weight"].float() + float(self.spec.weight_offset)).contiguous()
@@ -88,9 +90,14 @@ class WideRmsNorm(Norm):
         return self.rt.kernels.wide_rms_norm(x, self.weight, self.spec.eps, self.rt.dtype, None, None, rows)
 
     def add_norm(self, x: torch.Tensor, residual: torch.Tensor, rows: torch.Tensor | None = None, extra: torch.Tensor | None = None,
-                 gate: tuple | None = None):
+                 gate: tuple | None = None, post: "WideRmsNorm | None" = None):
         """Returns (norm(residual + x [+ extra]), the sum); without ``rows`` the sum replaces ``residual`` in place. ``gate``
-        (arguments: float32 like x, bias: float32 [hidden]): x is multiplied by sigmoid(arguments + bias) before it is added."""
+        (arguments: float32 like x, bias: float32 [hidden]): x is multiplied by sigmoid(arguments + bias) before it is added. ``post``: a
+        norm of its own that x passes before it is added, in the same kernel and never rounded between."""
+        if post is not None:
+            if extra is not None or gate is not None:
+                raise ValueError("rms_norm_wide: a normed addend takes neither a second addend nor a gate")
+            return self.rt.kernels.sandwich_norm(residual, x, post.weight, post.spec.eps, self.weight, self.spec.eps, rows), residual
         if gate is not None:
             if extra is not None:
                 raise ValueError("rms_norm_wide: a gated sum takes no second addend")

@@ -4,7 +4,7 @@ Per step: one fused q/k/v projection (rows [q heads | k heads | v heads], with a
 rotates the query and key heads (interleaved pairs or split halves, as the position encoding says; angles formed in double
 precision), divides each by its root mean square over the head (no weight), writes the query back in place and the key and
 value into the step's page slots; attention of the step's queries over the pages with p_j = exp(s_j) / (1 + sum exp(s_j)) (with
-``sink``; the plain softmax without), scores and weights in 32-bit, over every earlier key or the last ``window`` (the cache
+``sink``; exp(sink_h), a stored number a head, in the place of 1 with ``learned_sink``; the plain softmax without), scores and weights in 32-bit, over every earlier key or the last ``window`` (the cache
 group then gives back the pages the window has passed), a score s becoming c tanh(s / c) with ``softcap`` c; the output projection
 over the concatenated heads.
 
@@ -55,7 +55,11 @@ class SinkAttention(Mixer):
             raise ValueError(f"sink_attention: a window of {s.window} keys must be positive")
         if s.softcap < 0:
             raise ValueError(f"sink_attention: the scores' cap {s.softcap} cannot be negative")
+        if s.learned_sink and not s.sink:
+            raise ValueError("sink_attention: stored sinks belong to a softmax with a sink")
+        self.sinks = None
         self.halves = self.position is not None and getattr(self.position, "pairing", None) == "halves"
+        self.amplitude = getattr(self.position, "amplitude", 1.0)
         self.two_planes = s.head_dim == s.v_dim
 
     @classmethod
@@ -64,11 +68,15 @@ class SinkAttention(Mixer):
         decls = {"qkv": ParamDecl(shape=(Q + K + V, spec.hidden), row_splits=(Q, K, V)), "out": ParamDecl(shape=(spec.hidden, spec.num_heads * spec.v_dim))}
         if spec.bias:
             decls["qkv_bias"] = ParamDecl(shape=(Q + K + V,), row_splits=(Q, K, V), role="vector", init=("normal", 0.0, 0.1))
+        if spec.learned_sink:
+            decls["sink"] = ParamDecl(shape=(spec.num_heads,), role="vector", init=("normal", 0.0, 1.0))
         return decls
 
     def load(self, params):
         self.qkv.load(params["qkv"], params["qkv_bias"] if self.spec.bias else None)
         self.out.load(params["out"])
+        if self.spec.learned_sink:
+            self.sinks = params["sink"].float().contiguous()
 
     def cache_need(self) -> CacheNeed:
         s = self.spec
@@ -93,13 +101,14 @@ class SinkAttention(Mixer):
         q = torch.empty((qkv.shape[0], s.num_heads, s.head_dim), dtype=qkv.dtype, device=qkv.device) if tensor_cores else None
         k.sink_attention_prepare(qkv, cache.k_pool, cache.v_pool, inv_freq, rotary_dim, batch.positions, tables.slot_mapping, s.num_heads,
                                  s.num_kv_heads, s.head_dim, s.v_dim, s.unit_norm_eps, cache.page_size, **({"q_out": q} if tensor_cores else {}),
-                                 **({"halves": True} if self.halves else {}))
+                                 **({"halves": True} if self.halves else {}), **({"amplitude": self.amplitude} if self.amplitude != 1.0 else {}))
         if tensor_cores:
             o = self._attend_tensor_cores(q, batch, cache, tables)
         else:
             o = k.sink_attention(qkv, cache.k_pool, cache.v_pool, batch.positions, batch.token_row, tables.kv_indptr, tables.kv_indices,
                                  s.num_heads, s.num_kv_heads, s.head_dim, s.v_dim, s.scale, s.sink, kv_cap=batch.kv_cap,
-                                 **({"window": s.window} if s.window is not None else {}), **({"softcap": s.softcap} if s.softcap else {}))
+                                 **({"window": s.window} if s.window is not None else {}), **({"softcap": s.softcap} if s.softcap else {}),
+                                 **({"sinks": self.sinks} if self.sinks is not None else {}))
         return self.out(o)
 
     # ---- bfloat16 with keys and values of one size: the framework's tensor-core kernels, with the sink
@@ -111,7 +120,8 @@ class SinkAttention(Mixer):
         chunk, cluster = split_for(batch.num_rows, batch.kv_cap, cache.k_pool, cache.v_pool) if split_for and batch.kv_cap else (k.decode_chunk, 0)
         plan = batch.step_work(self, ("sink_attention", group, s.window, chunk, tile_rows, cluster))
         return k.attention_mma(q, cache.k_pool, cache.v_pool, batch.q_indptr, batch.kv_lens, tables.kv_indptr, tables.kv_indices, plan,
-                               s.scale, s.window, sink=s.sink, wide_weights=True, **({"softcap": s.softcap} if s.softcap else {}))
+                               s.scale, s.window, sink=s.sink, wide_weights=True, **({"softcap": s.softcap} if s.softcap else {}),
+                               **({"sinks": self.sinks} if self.sinks is not None else {}))
 
     def step_class(self, row_counts):
         return ("short_rows", any(n <= SHORT_ROW_TOKENS for n in row_counts))

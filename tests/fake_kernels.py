@@ -302,14 +302,14 @@ class FakeKernels:
 
     # ---- attention with a sink
     def sink_attention_prepare(self, qkv, k_pool, v_pool, inv_freq, rotary_dim, positions, slot_mapping, heads, kv_heads, dim, vdim, eps, page_size,
-                               halves=False):
+                               halves=False, q_out=None, amplitude=1.0):
         T = qkv.shape[0]
         Q, K = heads * dim, kv_heads * dim
 
         def turn(x):           # [T, n, dim] float32
             if rotary_dim:
                 ang = positions.double()[:, None] * inv_freq[None, :]
-                c, s = torch.cos(ang)[:, None, :].float(), torch.sin(ang)[:, None, :].float()
+                c, s = amplitude * torch.cos(ang)[:, None, :].float(), amplitude * torch.sin(ang)[:, None, :].float()
                 first, second = (slice(0, rotary_dim // 2), slice(rotary_dim // 2, rotary_dim)) if halves else (slice(0, rotary_dim, 2), slice(1, rotary_dim, 2))
                 u, v = x[..., first].clone(), x[..., second].clone()
                 x[..., first] = u * c - v * s
@@ -318,9 +318,13 @@ class FakeKernels:
                 x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
             return x
 
-        qkv[:, :Q] = turn(qkv[:, :Q].float().reshape(T, heads, dim)).reshape(T, Q).to(qkv.dtype)
-        k = turn(qkv[:, Q : Q + K].float().reshape(T, kv_heads, dim)).to(qkv.dtype)
-        v = qkv[:, Q + K :].reshape(T, kv_heads, vdim)
+        q = turn(qkv[:, :Q].float().reshape(T, heads, dim).clone()).to(qkv.dtype)
+        if q_out is not None:
+            q_out.copy_(q)
+        else:
+            qkv[:, :Q] = q.reshape(T, Q)
+        k = turn(qkv[:, Q : Q + K].float().reshape(T, kv_heads, dim).clone()).to(qkv.dtype)
+        v = qkv[:, Q + K : Q + K + kv_heads * vdim].reshape(T, kv_heads, vdim)
         for t in range(T):
             slot = int(slot_mapping[t])
             if slot < 0:
@@ -333,8 +337,69 @@ class FakeKernels:
                 k_pool[page, :, off, :] = k[t]
                 v_pool[page, :, off, :] = v[t]
 
+    @staticmethod
+    def _visible(k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, t, kv_heads, dim, vdim, window):
+        """(keys, values) float [kv_heads, n, .] that token t sees."""
+        page_size, pos, r = k_pool.shape[2], int(positions[t]), int(token_row[t])
+        pages = kv_indices[int(kv_indptr[r]) : int(kv_indptr[r + 1])].long()
+        lo = max(0, pos - window + 1) if window else 0
+        first_page = lo // page_size            # pages before it may have been given back (entry -1): never touched
+        pages, lo = pages[first_page : pos // page_size + 1], lo - first_page * page_size
+        hi = pos + 1 - first_page * page_size
+        assert (pages >= 0).all(), "a page inside the window was given back"
+        entries = k_pool[pages].permute(1, 0, 2, 3).reshape(kv_heads, -1, k_pool.shape[3])[:, lo:hi].float()
+        if v_pool is None:
+            return entries[..., :dim], entries[..., dim:]
+        return entries, v_pool[pages].permute(1, 0, 2, 3).reshape(kv_heads, -1, vdim)[:, lo:hi].float()
+
+    def talking_attention(self, q, out, k_pool, v_pool, gate, talk, positions, token_row, kv_indptr, kv_indices, kv_heads, vdim, scale, window=None,
+                          out_scale=1.0, kv_cap=0):
+        T, heads, dim = q.shape
+        group = heads // kv_heads
+        for t in range(T):
+            if int(positions[t]) < 0:
+                continue
+            keys, vals = self._visible(k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, t, kv_heads, dim, vdim, window)
+            own = torch.einsum("hd,hnd->hn", q[t].float(), keys.repeat_interleave(group, 0)) * scale
+            o = torch.einsum("hn,hnd->hd", torch.softmax(talk @ own, dim=-1), vals.repeat_interleave(group, 0)).reshape(-1) * out_scale
+            out[t] = (o * torch.sigmoid(gate[t].float()) if gate is not None else o).to(out.dtype)
+
+    # ---- the recurrence whose gates read only the current token
+    def min_gru_scan(self, u, out, z_bias, x_bias, out_scale, state, q_indptr, slots, width, chunked=None):
+        z = u[:, :width].float() + z_bias
+        x = u[:, width : 2 * width].float() + x_bias
+        g = u[:, 2 * width : 3 * width].float()
+        cand = torch.where(x >= 0, x + 0.5, torch.sigmoid(x))
+        for row in range(slots.numel()):
+            S = state[int(slots[row]), :width]
+            for t in range(int(q_indptr[row]), int(q_indptr[row + 1])):
+                S.copy_(torch.sigmoid(-z[t]) * S + torch.sigmoid(z[t]) * cand[t])
+                out[t] = (S * g[t] * torch.sigmoid(g[t]) * out_scale).to(out.dtype)
+
+    def retention_scan_raw(self, u, state, decay, q_indptr, slots, heads, dim, vdim, activation="none", k_scale=1.0, chunked=None):
+        act = torch.nn.functional.silu if activation == "silu" else (lambda z: z)
+        x = act(u[:, : heads * (2 * dim + vdim)].float())
+        qk = x[:, : 2 * heads * dim].clone()
+        qk[:, heads * dim :] *= k_scale
+        return self.retention_scan(qk, x, 2 * heads * dim, state, decay, q_indptr, slots, heads, dim, vdim)
+
+    def sandwich_norm(self, stream, addend, post_w, post_eps, w, eps, rows=None):
+        a = addend.float()
+        s = stream + a * torch.rsqrt((a * a).mean(-1, keepdim=True) + post_eps) * post_w
+        if rows is None:
+            stream.copy_(s)
+        else:
+            s = s[rows.long()]
+        return (s * torch.rsqrt((s * s).mean(-1, keepdim=True) + eps) * w).to(addend.dtype)
+
+    def weighted_sum(self, xs, ws):
+        return sum(float(w) * x.float() for w, x in zip(ws, xs)).to(xs[0].dtype)
+
+    def relu_squared(self, x):
+        return (torch.clamp(x.float(), min=0.0) ** 2).to(x.dtype)
+
     def sink_attention(self, qkv, k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, scale, sink, kv_cap=0,
-                       window=None, softcap=0.0):
+                       window=None, softcap=0.0, sinks=None):
         T = qkv.shape[0]
         page_size = k_pool.shape[2]
         out = torch.zeros(T, heads * vdim, dtype=qkv.dtype)
@@ -359,9 +424,10 @@ class FakeKernels:
                 s = (keys[h // group] @ q[h]) * scale
                 if softcap:
                     s = softcap * torch.tanh(s / softcap)
-                m = torch.clamp(s.max(), min=0.0) if sink else s.max()
+                at = sinks[h] if sinks is not None else torch.zeros(())
+                m = torch.maximum(s.max(), at) if sink else s.max()
                 e = torch.exp(s - m)
-                out[t, h * vdim : (h + 1) * vdim] = ((e / (e.sum() + (torch.exp(-m) if sink else 0.0))) @ vals[h // group]).to(qkv.dtype)
+                out[t, h * vdim : (h + 1) * vdim] = ((e / (e.sum() + (torch.exp(at - m) if sink else 0.0))) @ vals[h // group]).to(qkv.dtype)
         return out
 
     # ---- a 32-bit stream with root-mean-square norms, a hashed pair embedding, token inputs
