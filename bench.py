@@ -576,6 +576,63 @@ def lovurax_main(args) -> int:
     return 0
 
 
+# Revirax models at the same widths, depths and vocabularies, every layer with a feed-forward of 4 x width without a gate: of every four
+# layers one holds a windowed attention that mixes its scores across the heads (16 query heads over 4 key/value heads) beside a recurrence
+# as wide as the model, one a retention over activated projections (heads of 64 keys and 128 values, as wide in values as the model), two
+# an attention with a stored sink a head over every earlier key. The Nomivik model beside each is the closest design the engine has (a
+# 32-bit stream, a windowed attention beside a recurrence with a matrix state, gated recurrences).
+def _revirax_config(width, heads, dim, layers, vocab, window, **_):
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": window},
+            "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    parallel = {"type": "parallel", "mixer": {"left": left, "right": {"width": width}, "left_scale": 0.7, "right_scale": 0.9}}
+    lightning = {"type": "lightning", "mixer": {"heads": width // 128, "dim": 64, "vdim": 128,
+                                                "decay": [1.0 - 2.0 ** (-5 - 3 * h / max(width // 128 - 1, 1)) for h in range(width // 128)]}}
+    attention = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                "rot": {"base": 500000.0, "dims": dim,
+                                                        "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}}
+    order = (parallel, attention, lightning, attention)
+    return {"architecture": "Revirax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "layers": [dict(order[i % 4], mlp={"kind": "dense", "ff": 4 * width}) for i in range(layers)]}
+
+
+def revirax_main(args) -> int:
+    """Prefill and decode throughput of Revirax models beside Nomivik models (the closest design the engine has) of equal width,
+    depth and vocabulary, one JSON line."""
+    import torch
+
+    from roost_b200.config.nomivik import NomivikConfig
+    from roost_b200.config.revirax import ReviraxConfig
+    pk, pk_src = peaks()
+    out = {}
+    for name in args.design_sizes.split(","):
+        s = dict(DESIGN_SIZES[name])
+        s["dim"] = 128 if s["width"] >= 2048 else 64
+        s["dense_ff"] = 3 * s["width"]
+        rec = {}
+        for which in ("revirax", "nomivik"):
+            if which == "revirax":
+                model, _ = build_from_config(ReviraxConfig, _revirax_config(**s), torch.bfloat16)
+            else:
+                model, _ = build_from_config(NomivikConfig, _nomivik_config(**s), torch.bfloat16)
+            r = {"weight_gb": round(model.weight_bytes() / 1e9, 3)}
+            ms = timed_prefill(model, args.prefill_tokens)
+            r["prefill"] = {"tokens": args.prefill_tokens, "ms": round(ms, 3), "tokens_per_s": round(args.prefill_tokens / ms * 1e3)}
+            for batch in _ints(args.design_batches):
+                tps, ms, launches, _ = timed_decode(model, batch, args.design_context, args.steps, max(args.warmup, 3))
+                r[f"decode_b{batch}"] = {"context": args.design_context, "ms": round(ms, 4), "tokens_per_s": round(tps), "launches": launches[0] // args.steps,
+                                         "library_launches": launches[1] // args.steps}
+            rec[which] = r
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        rec["config"] = {k: s[k] for k in ("width", "heads", "dim", "layers", "vocab", "window")}
+        out[name] = rec
+    print(json.dumps({"metric": "prefill and decode tokens/s of Revirax models beside Nomivik models of equal width, depth and vocabulary",
+                      "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "impl": "ours", "peaks": pk_src,
+                      "data": "synthetic: seeded random weights, seeded random tokens; device-timed with CUDA events", "sizes": out}))
+    return 0
+
+
 def designs_main(args) -> int:
     """Prefill and decode throughput of Vamatar models beside Qwen3-shaped models of equal size, one JSON line."""
     import torch
@@ -585,6 +642,8 @@ def designs_main(args) -> int:
         return nomivik_main(args)
     if args.design == "lovurax":
         return lovurax_main(args)
+    if args.design == "revirax":
+        return revirax_main(args)
     pk, pk_src = peaks()
     out = {}
     for name in args.design_sizes.split(","):
@@ -633,9 +692,9 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="layers built (default: all the layers of --sizes)")
     ap.add_argument("--sizes", default="8b", choices=sorted(SIZES), help="whose layer sizes: Qwen3-0.6B, -8B (the headline) or -32B")
     ap.add_argument("--design-sizes", default="w1024,w2048", help="--workload designs: which of the Vamatar layer sizes to measure")
-    ap.add_argument("--design", default="vamatar", choices=["vamatar", "lafanex", "nomivik", "lovurax"],
+    ap.add_argument("--design", default="vamatar", choices=["vamatar", "lafanex", "nomivik", "lovurax", "revirax"],
                     help="--workload designs: vamatar (beside Qwen3-shaped models), lafanex (beside Vamatar models of equal size) or "
-                         "nomivik (beside Lafanex models with dense feed-forwards of equal size) or lovurax (beside Nomivik models of "
+                         "nomivik (beside Lafanex models with dense feed-forwards of equal size) or lovurax or revirax (beside Nomivik models of "
                          "equal size)")
     ap.add_argument("--design-batches", default="1,8", help="--workload designs: decode batch sizes")
     ap.add_argument("--design-context", type=int, default=1024, help="--workload designs: keys every decoding request holds")
