@@ -13,6 +13,7 @@
 // shared memory (beyond); a token's (k, q) are staged in shared memory once and read by all lanes; the next token's inputs are
 // loaded while the current one is multiplied. Where nothing is rotated the scan reads the projection's row [q heads | k heads | v heads]
 // itself (RAW): q, k and v pass SiLU (act 1) or stay as they are, k is multiplied by k_scale, all in 32-bit, and no prepare kernel runs.
+// In chunks (two walks, a block a slice of 32 columns) that repeats the activations; there the prepare kernel applies them once to q and k.
 //
 // Steps of many tokens cut every row into chunks of 64 tokens that run side by side (three launches): a chunk of n tokens walked
 // from S = 0 ends with S'; a state S before the chunk is decay^n S + S' after it. The first walk leaves every chunk's own S', one
@@ -27,14 +28,14 @@ constexpr int kRtChunkTokens = 64;
 template <typename T>
 __global__ void __launch_bounds__(128) retention_prepare_kernel(const T* __restrict__ u, int64_t ld, float* __restrict__ qk,
                                                                const double* __restrict__ inv_freq, const int32_t* __restrict__ positions,
-                                                               int heads, int dim, int rot_dims, float k_scale) {
+                                                               int heads, int dim, int rot_dims, float k_scale, int act) {
   extern __shared__ float sm[];      // rot_dims/2 cosines, rot_dims/2 sines
   const int half = rot_dims / 2;
   float* cs = sm;
   float* sn = sm + half;
   pdl_launch_dependents();
   const int t = blockIdx.x;
-  const int pos = positions[t];
+  const int pos = half > 0 ? positions[t] : 0;
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
     double ang = (double)pos * inv_freq[i];
     ang -= 6.283185307179586476925286766559 * rint(ang * 0.15915494309189533576888376337251);
@@ -48,7 +49,7 @@ __global__ void __launch_bounds__(128) retention_prepare_kernel(const T* __restr
   for (int idx = threadIdx.x; idx < n; idx += blockDim.x) {
     const int j = idx % dim;
     const float x = to_float(row[idx]);
-    float y = x;
+    float y = act ? silu_f(x) : x;
     if (j < half) {
       y = x * cs[j] - to_float(row[idx + half]) * sn[j];
     } else if (j < rot_dims) {
@@ -144,7 +145,7 @@ __global__ void __launch_bounds__(32) retention_scan_kernel(const void* __restri
       const int d = lane + 32 * i;
       if (d < dim) stage[d] = !RAW ? make_float2(nk[i], nq[i]) : (act ? make_float2(silu_f(nk[i]) * k_scale, silu_f(nq[i])) : make_float2(nk[i] * k_scale, nq[i]));
     }
-    const float val = RAW && act ? silu_f(nv) : nv;
+    const float val = act ? silu_f(nv) : nv;
     if (t + 1 < end) load(t + 1);
     __syncwarp();
     float num = 0.f;
@@ -221,16 +222,17 @@ __global__ void retention_carry_kernel(const float* state, int64_t state_stride,
 using namespace roost;
 
 extern "C" int roost_retention_prepare(const void* u, int64_t ld, float* qk, const double* inv_freq, const int32_t* positions, int tokens, int heads,
-                                       int dim, int rot_dims, float k_scale, int dtype, roost_stream_t stream) {
+                                       int dim, int rot_dims, float k_scale, int act, int dtype, roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && dim > 0, "retention_prepare: sizes must be positive");
   ROOST_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim, "retention_prepare: the rotated width must be even and at most dim");
-  ROOST_REQUIRE(u && qk && positions && (rot_dims == 0 || inv_freq), "retention_prepare: a pointer is null");
+  ROOST_REQUIRE(u && qk && (rot_dims == 0 || (inv_freq && positions)), "retention_prepare: a pointer is null");
   ROOST_REQUIRE(ld >= (int64_t)2 * heads * dim, "retention_prepare: a row is too narrow");
+  ROOST_REQUIRE(act == 0 || (act == 1 && rot_dims == 0), "retention_prepare: the activation is none (0) or, without a rotation, SiLU (1)");
   if (tokens == 0) return ROOST_OK;
   const size_t smem = ((size_t)rot_dims + 2) * sizeof(float);
   if (smem > 48 * 1024) return fail(ROOST_ERR_UNSUPPORTED, "retention_prepare: a rotation of more than 12286 elements");
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(retention_prepare_kernel<T>, dim3(tokens), dim3(128), smem, (cudaStream_t)stream, (const T*)u, ld, qk,
-                                               inv_freq, positions, heads, dim, rot_dims, k_scale));
+                                               inv_freq, positions, heads, dim, rot_dims, k_scale, act));
   return check_launch("retention_prepare");
 }
 
@@ -277,15 +279,15 @@ static int retention_scan_launch(const void* qk, int64_t ldqk, int act, float k_
 // ws (float[chunks * heads * dim * vdim], chunks = roost_retention_scan_chunks(tokens, rows)): rows are cut into chunks that run side
 // by side (three launches); null: every row is walked in one pass.
 extern "C" int roost_retention_scan(const float* qk, const void* v, int64_t ldv, float* out, float* state, int64_t state_stride, const float* decay,
-                                    const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, float* ws,
-                                    int dtype, roost_stream_t stream) {
-  ROOST_REQUIRE(rows >= 0 && tokens >= 0 && heads > 0 && dim > 0 && vdim > 0, "retention_scan: sizes must be positive");
+                                    const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, int v_act,
+                                    float* ws, int dtype, roost_stream_t stream) {
+  ROOST_REQUIRE(rows >= 0 && tokens >= 0 && heads > 0 && dim > 0 && vdim > 0 && (v_act == 0 || v_act == 1), "retention_scan: sizes must be positive");
   ROOST_REQUIRE(qk && v && out && state && decay && q_indptr && slots, "retention_scan: a pointer is null");
   ROOST_REQUIRE(ldv >= (int64_t)heads * vdim && state_stride >= (int64_t)heads * dim * vdim, "retention_scan: a row or a slot is too narrow");
   if (dim > 1024) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan: heads of more than 1024 keys");
   if (heads > 65535 || (vdim + 31) / 32 > 65535) return fail(ROOST_ERR_UNSUPPORTED, "retention_scan: too many heads or values");
   if (rows == 0 || tokens == 0) return ROOST_OK;
-  ROOST_DISPATCH_DTYPE(dtype, T, return (retention_scan_launch<T, false>(qk, 0, 0, 1.0f, (const T*)v, ldv, out, state, state_stride, decay, q_indptr, slots,
+  ROOST_DISPATCH_DTYPE(dtype, T, return (retention_scan_launch<T, false>(qk, 0, v_act, 1.0f, (const T*)v, ldv, out, state, state_stride, decay, q_indptr, slots,
                                                                          rows, tokens, heads, dim, vdim, ws, (cudaStream_t)stream)));
 }
 

@@ -452,15 +452,16 @@ int roost_head_norm_gate(const float* o, const void* u, int64_t ld_u, int col, c
                          float eps, int gate_silu, int dtype, roost_stream_t stream);
 
 /* ---- retention (retention.cu): S <- decay_h S + k v^T, o = S^T q a head; the slot holds S [heads, dim, vdim] ---- */
-/* qk (float32 [tokens, 2 * heads * dim]) = the rotated query heads and the rotated, scaled key heads of rows [q heads | k heads | ...]. */
+/* qk (float32 [tokens, 2 * heads * dim]) = the rotated query heads and the rotated, scaled key heads of rows [q heads | k heads | ...]; act 1
+ * (without a rotation): SiLU of both. */
 int roost_retention_prepare(const void* u, int64_t ld, float* qk, const double* inv_freq, const int32_t* positions, int tokens, int heads,
-                            int dim, int rot_dims, float k_scale, int dtype, roost_stream_t stream);
+                            int dim, int rot_dims, float k_scale, int act, int dtype, roost_stream_t stream);
 /* ws: float[roost_retention_scan_chunks(tokens, rows) * heads * dim * vdim], or null. With it the rows are cut into chunks of 64 tokens
- * that run side by side. v: the values' first column in rows ldv apart; out float32 [tokens, heads * vdim]. */
+ * that run side by side. v: the values' first column in rows ldv apart (v_act 1: SiLU of them); out float32 [tokens, heads * vdim]. */
 int roost_retention_scan_chunks(int tokens, int rows);
 int roost_retention_scan(const float* qk, const void* v, int64_t ldv, float* out, float* state, int64_t state_stride, const float* decay,
-                         const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, float* ws, int dtype,
-                         roost_stream_t stream);
+                         const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, int v_act, float* ws,
+                         int dtype, roost_stream_t stream);
 
 /* The same where nothing is rotated, over the projection's rows u = [q heads | k heads | v heads | ...], ld apart: act 1 puts SiLU on q, k
  * and v (0: nothing), the keys are multiplied by k_scale. */
@@ -490,6 +491,18 @@ int roost_talking_attention(const void* q, void* out, int64_t ld_out, float* par
                             const int32_t* kv_indptr, const int32_t* kv_indices, int tokens, int heads, int kv_heads, int dim, int vdim,
                             int page_size, float scale, int window, float out_scale, int key_tile, int splits, int tiles_per_split, int dtype,
                             roost_stream_t stream);
+
+/* The same on the tensor cores (talking_attention_mma.cu; bfloat16, dim a multiple of 16, vdim too and at most 128, whatever fits the shared
+ * memory), a block per (row, 16 query tokens, range of output heads): for steps that bring prompt portions. talk holds numbers that are exact
+ * in bfloat16. q_indptr: the rows' token ranges (rows + 1 entries). */
+int roost_talking_attention_mma_supported(int heads, int kv_heads, int dim, int vdim, int entry);
+int roost_talking_attention_mma(const void* q, void* out, int64_t ld_out, const void* k_base, const void* v_base, int entry, const void* gate,
+                                int64_t ld_gate, const float* talk, const int32_t* positions, const int32_t* q_indptr, const int32_t* kv_indptr,
+                                const int32_t* kv_indices, int tokens, int rows, int heads, int kv_heads, int dim, int vdim, int page_size,
+                                float scale, int window, float out_scale, const int32_t* token_row, float* ws, int tiles_a_chunk, int max_chunks,
+                                roost_stream_t stream);   /* max_chunks > 1: a tile's keys in chunks of tiles_a_chunk tiles of 32 keys, their sums in
+                                                             ws: float[tokens * heads * max_chunks * (vdim + 2)], combined by a second kernel; the
+                                                             last chunk takes what a longer row has left */
 
 /* ---- attention with sigmoid weights (sigmoid_attention.cu) ---- */
 /* Queries and keys divided by their root mean square times q_w / k_w (dim numbers each); queries times

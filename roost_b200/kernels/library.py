@@ -168,10 +168,10 @@ _SIGNATURES = {
     "roost_matrix_memory_scan": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                  c_float, c_float, c_void_p, c_int, c_void_p],
     "roost_head_norm_gate": [c_void_p, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
-    "roost_retention_prepare": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    "roost_retention_prepare": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
     "roost_retention_scan_chunks": [c_int, c_int],
     "roost_retention_scan": [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                             c_void_p, c_int, c_void_p],
+                             c_int, c_void_p, c_int, c_void_p],
     "roost_sigmoid_attention_prepare": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                         c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_void_p],
     "roost_sigmoid_attention": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -192,6 +192,10 @@ _SIGNATURES = {
     "roost_talking_attention": [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_int, c_int, c_int, c_int,
                                 c_void_p],
+    "roost_talking_attention_mma_supported": [c_int, c_int, c_int, c_int, c_int],
+    "roost_talking_attention_mma": [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int,
+                                    c_void_p],
     "roost_relu_squared": [c_void_p, c_void_p, c_int64, c_int, c_void_p],
     "roost_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "roost_weighted_sum": [c_void_p, c_void_p, c_int, c_void_p, c_int64, c_int, c_void_p],
@@ -1163,24 +1167,26 @@ class KernelLibrary:
         return out
 
     # ------------------------------------------------------------------ retention
-    def retention_prepare(self, u, inv_freq, rotary_dim: int, positions, heads: int, dim: int, k_scale: float) -> torch.Tensor:
-        """The rotated query heads and the rotated, scaled key heads of rows [q heads | k heads | ...] as float32 [T, 2 * heads * dim]."""
-        _need(u, "u"); _need(positions, "positions", torch.int32)
+    def retention_prepare(self, u, inv_freq, rotary_dim: int, positions, heads: int, dim: int, k_scale: float, activation: str = "none") -> torch.Tensor:
+        """The rotated query heads and the rotated, scaled key heads of rows [q heads | k heads | ...] as float32 [T, 2 * heads * dim];
+        ``activation`` "silu" (without a rotation): SiLU of both."""
+        _need(u, "u")
         if rotary_dim:
-            _need(inv_freq, "inv_freq", torch.float64)
+            _need(positions, "positions", torch.int32); _need(inv_freq, "inv_freq", torch.float64)
             if inv_freq.numel() != rotary_dim // 2:
                 raise KernelError("retention_prepare: inv_freq must have rotary_dim / 2 entries")
         T = u.shape[0]
         if u.shape[1] < 2 * heads * dim:
             raise KernelError("retention_prepare: the rows do not hold the query and key heads")
         qk = torch.empty((T, 2 * heads * dim), dtype=torch.float32, device=u.device)
-        self._call("roost_retention_prepare", _ptr(u), u.stride(0), _ptr(qk), _ptr(inv_freq) if rotary_dim else None, _ptr(positions), T, heads, dim,
-                   rotary_dim, float(k_scale), dtype_code(u.dtype), _stream())
+        self._call("roost_retention_prepare", _ptr(u), u.stride(0), _ptr(qk), _ptr(inv_freq) if rotary_dim else None, _ptr(positions) if rotary_dim else None, T,
+                   heads, dim, rotary_dim, float(k_scale), 1 if activation == "silu" else 0, dtype_code(u.dtype), _stream())
         return qk
 
-    def retention_scan(self, qk, u, v_col: int, state, decay, q_indptr, slots, heads: int, dim: int, vdim: int, chunked: bool | None = None) -> torch.Tensor:
+    def retention_scan(self, qk, u, v_col: int, state, decay, q_indptr, slots, heads: int, dim: int, vdim: int, chunked: bool | None = None,
+                       activation: str = "none") -> torch.Tensor:
         """S <- decay_h S + k v^T, o = S^T q a head: float32 [T, heads * vdim]; see csrc/retention.cu. The values are the columns
-        from ``v_col`` on of ``u``. ``chunked`` None: steps of ``SCAN_CHUNKED_MIN_TOKENS`` tokens or more cut their rows into chunks."""
+        from ``v_col`` on of ``u`` (``activation`` "silu": their SiLU). ``chunked`` None: steps of ``SCAN_CHUNKED_MIN_TOKENS`` tokens or more cut their rows into chunks."""
         _need(qk, "qk", torch.float32); _need(u, "u"); _need(state, "state", torch.float32); _need(decay, "decay", torch.float32)
         _need(q_indptr, "q_indptr", torch.int32); _need(slots, "slots", torch.int32)
         T = u.shape[0]
@@ -1192,14 +1198,15 @@ class KernelLibrary:
             chunks = self._lib.roost_retention_scan_chunks(T, slots.numel())
             ws = torch.empty((chunks * heads * dim * vdim,), dtype=torch.float32, device=u.device)
         self._call("roost_retention_scan", _ptr(qk), u.data_ptr() + v_col * u.element_size(), u.stride(0), _ptr(out), _ptr(state), state.stride(0),
-                   _ptr(decay), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, _ptr(ws), dtype_code(u.dtype), _stream(),
-                   launches=3 if ws is not None else 1)
+                   _ptr(decay), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, 1 if activation == "silu" else 0, _ptr(ws),
+                   dtype_code(u.dtype), _stream(), launches=3 if ws is not None else 1)
         return out
 
     def retention_scan_raw(self, u, state, decay, q_indptr, slots, heads: int, dim: int, vdim: int, activation: str = "none", k_scale: float = 1.0,
                            chunked: bool | None = None) -> torch.Tensor:
         """The same where nothing is rotated, over the projection's rows ``u`` = [q heads | k heads | v heads | ...]: ``activation`` "silu"
-        puts SiLU on q, k and v, the keys are multiplied by ``k_scale``."""
+        puts SiLU on q, k and v, the keys are multiplied by ``k_scale``. Rows that are cut into chunks are walked twice, a block a slice of
+        the values' columns: there the activations of q and k are made once, by the prepare kernel."""
         if activation not in ("none", "silu"):
             raise KernelError(f"retention_scan_raw: activation '{activation}' is neither none nor silu")
         _need_rows(u, "u"); _need(state, "state", torch.float32); _need(decay, "decay", torch.float32)
@@ -1207,11 +1214,11 @@ class KernelLibrary:
         T = u.shape[0]
         if u.shape[1] < heads * (2 * dim + vdim) or decay.numel() != heads:
             raise KernelError("retention_scan_raw: the rows or the decays do not fit the sizes")
+        if ((T >= self.SCAN_CHUNKED_MIN_TOKENS) if chunked is None else chunked) and u.is_contiguous():
+            qk = self.retention_prepare(u, None, 0, None, heads, dim, k_scale, activation=activation)
+            return self.retention_scan(qk, u, 2 * heads * dim, state, decay, q_indptr, slots, heads, dim, vdim, chunked=True, activation=activation)
         out = torch.empty((T, heads * vdim), dtype=torch.float32, device=u.device)
         ws = None
-        if (T >= self.SCAN_CHUNKED_MIN_TOKENS) if chunked is None else chunked:
-            chunks = self._lib.roost_retention_scan_chunks(T, slots.numel())
-            ws = torch.empty((chunks * heads * dim * vdim,), dtype=torch.float32, device=u.device)
         self._call("roost_retention_scan_raw", _ptr(u), u.stride(0), 1 if activation == "silu" else 0, float(k_scale), _ptr(out), _ptr(state),
                    state.stride(0), _ptr(decay), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, _ptr(ws), dtype_code(u.dtype), _stream(),
                    launches=3 if ws is not None else 1)
@@ -1251,10 +1258,19 @@ class KernelLibrary:
         per = -(-tiles // splits)
         return -(-tiles // per), per
 
+    TALKING_MMA_MIN_TOKENS = 32     # tokens from which a bfloat16 step that brings prompt portions runs the tensor-core form
+    TALKING_MMA_CHUNK_TILES = 12    # tiles of 32 keys a block of the tensor-core form takes of a tile of queries
+
+    def talking_attention_mma_supported(self, heads: int, kv_heads: int, dim: int, vdim: int, two_planes: bool) -> bool:
+        return bool(self._lib.roost_talking_attention_mma_supported(heads, kv_heads, dim, vdim, dim if two_planes else dim + vdim))
+
     def talking_attention(self, q, out, k_pool, v_pool, gate, talk, positions, token_row, kv_indptr, kv_indices, kv_heads: int, vdim: int, scale: float,
-                          window: int | None = None, out_scale: float = 1.0, kv_cap: int = 0) -> None:
+                          window: int | None = None, out_scale: float = 1.0, kv_cap: int = 0, q_indptr: torch.Tensor | None = None) -> None:
         """Attention of the prepared queries q [T, heads, dim] whose scores are mixed across the heads by ``talk`` [heads, heads] before the
-        softmax, times sigmoid(``gate``) (rows may lie apart; None: no gate) and ``out_scale``, into ``out`` [T, heads * vdim]."""
+        softmax, times sigmoid(``gate``) (rows may lie apart; None: no gate) and ``out_scale``, into ``out`` [T, heads * vdim]. With
+        ``q_indptr`` (the rows' token ranges; ``talk`` then holds numbers that are exact in bfloat16) a bfloat16 step runs on the tensor cores
+        where the sizes and alignments allow; without, the 32-bit form, a token's keys dealt to several blocks when the step alone would not
+        fill the device."""
         _need(q, "q"); _need_rows(out, "out", q.dtype); _need(k_pool, "k_pool", q.dtype); _need(talk, "talk", torch.float32)
         for n, t in (("positions", positions), ("token_row", token_row), ("kv_indptr", kv_indptr), ("kv_indices", kv_indices)):
             _need(t, n, torch.int32)
@@ -1266,6 +1282,21 @@ class KernelLibrary:
         if tuple(out.shape) != (T, heads * vdim) or tuple(talk.shape) != (heads, heads):
             raise KernelError("talking_attention: out or the mixing matrix do not fit the sizes")
         kb, vb, entry = self._sink_cache(k_pool, v_pool, dim, vdim)
+        if (q_indptr is not None and q.dtype == torch.bfloat16 and self.talking_attention_mma_supported(heads, kv_heads, dim, vdim, v_pool is not None)
+                and out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0
+                and (gate is None or (gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0))):
+            _need(q_indptr, "q_indptr", torch.int32)
+            # a tile of queries with more than TALKING_MMA_CHUNK_TILES tiles of keys has them dealt to several blocks; the bound on the
+            # requests' lengths and the window say how many (every replay of a captured step agrees). 16 queries span window + 15 keys.
+            per = self.TALKING_MMA_CHUNK_TILES
+            span = min(kv_cap, window + 15 + 62) if (window and kv_cap) else kv_cap
+            max_chunks = max(1, -(-(-(-span // 32)) // per))
+            ws = torch.empty((T * heads * max_chunks * (vdim + 2),), dtype=torch.float32, device=q.device) if max_chunks > 1 else None
+            self._call("roost_talking_attention_mma", _ptr(q), _ptr(out), out.stride(0), kb, vb, entry, _ptr(gate), gate.stride(0) if gate is not None else 0,
+                       _ptr(talk), _ptr(positions), _ptr(q_indptr), _ptr(kv_indptr), _ptr(kv_indices), T, q_indptr.numel() - 1, heads, kv_heads, dim, vdim,
+                       k_pool.shape[2], float(scale), int(window or 0), float(out_scale), _ptr(token_row), _ptr(ws), per, max_chunks, _stream(),
+                       launches=2 if max_chunks > 1 else 1)
+            return
         kt = self.talking_key_tile(heads, kv_heads, dim, vdim, q.dtype)
         # a window's keys span at most window + key_tile - 1 positions' worth of tiles, whatever the requests' lengths are
         span = min(kv_cap, window + 2 * kt - 2) if (window and kv_cap) else kv_cap

@@ -52,6 +52,7 @@ class TalkingAttention(Mixer):
         self.amplitude = getattr(self.position, "amplitude", 1.0)
         self.two_planes = s.head_dim == s.v_dim
         self.talk = None
+        self.talk_exact = False
 
     @classmethod
     def parameters(cls, spec: TalkingAttentionSpec):
@@ -78,6 +79,8 @@ class TalkingAttention(Mixer):
 
     def load_middle(self, params):
         self.talk = params["talk"].float().contiguous()
+        # the tensor-core form takes the matrix as one bfloat16 operand: only where nothing of it is lost
+        self.talk_exact = bool((self.talk.to(torch.bfloat16).float() == self.talk).all())
 
     def load(self, params):
         self.proj_in.load(*self.input_weight(params))
@@ -98,8 +101,12 @@ class TalkingAttention(Mixer):
         k.sink_attention_prepare(u, cache.k_pool, cache.v_pool, inv_freq, rotary_dim, batch.positions, tables.slot_mapping, s.num_heads,
                                  s.num_kv_heads, s.head_dim, s.v_dim, None, cache.page_size, q_out=q, halves=self.halves, amplitude=self.amplitude)
         gate = u[:, self.qkv_width : self.in_width] if s.output_gate else None
+        # steps that bring prompt portions run on the tensor cores in bfloat16 where the sizes allow (a function of the step's size
+        # and kind only, so a captured step keeps its way); steps that decode, float32 and other sizes run the 32-bit kernel
+        portions = self.talk_exact and not batch.all_single and batch.num_tokens >= getattr(k, "TALKING_MMA_MIN_TOKENS", 1 << 30)
         k.talking_attention(q, out, cache.k_pool, cache.v_pool, gate, self.talk, batch.positions, batch.token_row, tables.kv_indptr, tables.kv_indices,
-                            s.num_kv_heads, s.v_dim, s.scale, window=s.window, out_scale=scale, kv_cap=batch.kv_cap)
+                            s.num_kv_heads, s.v_dim, s.scale, window=s.window, out_scale=scale, kv_cap=batch.kv_cap,
+                            **({"q_indptr": batch.q_indptr} if portions else {}))
 
     def __call__(self, x, batch, cache, write_cache: bool = True):
         if not write_cache:

@@ -535,7 +535,7 @@ class FakeKernels:
         return (x * torch.sigmoid(g) * (g if gate == "silu" else 1.0)).to(out_dtype)
 
     # ---- retention
-    def retention_prepare(self, u, inv_freq, rotary_dim, positions, heads, dim, k_scale):
+    def retention_prepare(self, u, inv_freq, rotary_dim, positions, heads, dim, k_scale, activation="none"):
         T = u.shape[0]
         x = u[:, : 2 * heads * dim].float().reshape(T, 2 * heads, dim).clone()
         if rotary_dim:
