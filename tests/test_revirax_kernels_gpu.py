@@ -175,7 +175,7 @@ def test_the_attention_with_a_stored_sink_a_head(kernels, dtype, heads, kv_heads
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("width", [1, 37, 320])
+@pytest.mark.parametrize("width", [1, 37, 288])
 @pytest.mark.parametrize("chunked", [False, True])
 def test_the_recurrence_whose_gates_read_only_the_current_token(kernels, dtype, width, chunked):
     g = torch.Generator().manual_seed(width)
