@@ -1,7 +1,7 @@
 """The cache manager: which pages and state slots every live request holds.
 
 Runs of mixers are sorted into groups by what they keep between steps (``CacheNeed``): paged keys and values
-of one geometry with every earlier token, paged with a window, or a fixed-size state per request. Each paged
+of one geometry with every earlier token, paged with a window (possibly beside the request's first tokens), or a fixed-size state per request. Each paged
 group has a pool of page ids of its own and a block table per request (index = position // page size; a page
 that a window has passed is given back and its entry becomes ``NULL_PAGE``); one page id addresses the page of
 every run in the group. Each state group has a pool of slots, one per live request. The reference's state
@@ -36,6 +36,7 @@ class CacheGroup:
     planes: int = 2                # tensors kept per token: keys and values, or one
     state_shape: tuple = ()
     state_dtype: torch.dtype = torch.float32
+    keep_first: int = 0            # with a window: the request's first tokens, which stay visible and whose pages are never given back
 
     def bytes_per_page(self, element_size: int) -> int:
         return self.planes * len(self.runs) * self.page_size * self.kv_heads * self.head_dim * element_size
@@ -151,7 +152,7 @@ class CacheManager:
                 continue
             table = rc.tables[gi]
             n = min(leading_releasable_pages(new_total, g.window, g.page_size), len(table))
-            for i in range(n):
+            for i in range(-(-g.keep_first // g.page_size), n):
                 if table[i] != NULL_PAGE:
                     self.pools[gi].release(table[i])
                     table[i] = NULL_PAGE
@@ -201,7 +202,7 @@ def build_groups(needs: list, page_size: int) -> list[CacheGroup]:
     """Sorts the schedule's runs into groups. ``needs[i]`` is the ``CacheNeed`` of run i, or None when the run
     keeps nothing or reads another run's cache; a tuple of them for a run whose mixer is several side by side (branch j's
     cache is then known as (i, j)). ``needs`` may also be a dict from any such key to its need (the embedding's state goes
-    under a key of its own). Paged runs with the same (window, kv_heads, head_dim, planes) share a
+    under a key of its own). Paged runs with the same (window, kv_heads, head_dim, planes, keep_first) share a
     group; every state run with the same shape and dtype shares one. A group of fixed-size state always exists,
     with no runs and a zero-sized state when the model has none, so that slots are handed out and returned on
     every path."""
@@ -219,16 +220,18 @@ def build_groups(needs: list, page_size: int) -> list[CacheGroup]:
         if need.kind == "paged":
             if need.planes not in (1, 2):
                 raise ValueError(f"run {i} asks for {need.planes} tensors a token; a paged cache keeps 1 or 2")
-            paged.setdefault((need.window, need.kv_heads, need.head_dim, need.planes), []).append(i)
+            if need.keep_first < 0 or (need.keep_first and need.window is None):
+                raise ValueError(f"run {i} keeps its first {need.keep_first} tokens: that belongs to a window")
+            paged.setdefault((need.window, need.kv_heads, need.head_dim, need.planes, need.keep_first), []).append(i)
         elif need.kind == "state":
             state.setdefault((tuple(need.state_shape), need.state_dtype), []).append(i)
         else:
             raise ValueError(f"run {i} asks for a cache of kind '{need.kind}'")
     groups = []
-    for (window, kvh, d, planes), runs in paged.items():
-        name = ("full" if window is None else f"window{window}") + f"_h{kvh}d{d}" + ("" if planes == 2 else f"x{planes}")
+    for (window, kvh, d, planes, keep_first), runs in paged.items():
+        name = ("full" if window is None else f"window{window}" + (f"keep{keep_first}" if keep_first else "")) + f"_h{kvh}d{d}" + ("" if planes == 2 else f"x{planes}")
         groups.append(CacheGroup(name=name, kind="paged", runs=tuple(runs), page_size=page_size, window=window,
-                                 kv_heads=kvh, head_dim=d, planes=planes))
+                                 kv_heads=kvh, head_dim=d, planes=planes, keep_first=keep_first))
     for (shape, dt), runs in state.items():
         groups.append(CacheGroup(name="state" + "x".join(map(str, shape)), kind="state", runs=tuple(runs),
                                  state_shape=shape, state_dtype=dt))

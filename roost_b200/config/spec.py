@@ -83,7 +83,9 @@ class LatentAttentionSpec(MixerSpec):
     (None: all). ``own_latent`` False: the run makes no latent and reads another run's; ``cache_window`` is then the
     window the shared cache is kept for (the widest of the runs that read it; None: everything is kept). ``rope_dim`` 0 (and no
     ``position``): keys have no rotated part and the cache entry is the latent alone. ``head_gate``: head h's output is multiplied
-    by sigmoid((W_g x)_h), one number a token and head, from the mixer's own input."""
+    by sigmoid((W_g x)_h), one number a token and head, from the mixer's own input. ``q_rank`` > 0: queries go through a latent of their own,
+    q = W_uq n(W_dq x) with n a root-mean-square norm (``latent_eps``, a stored weight). ``learned_sink``: the softmax's denominator also
+    holds exp(sink_h), a stored number a head. ``output_gate``: the heads side by side are multiplied element by element by sigmoid(W_g x)."""
     kind: str = "latent_attention"
     hidden: int = 0
     num_heads: int = 0
@@ -98,6 +100,9 @@ class LatentAttentionSpec(MixerSpec):
     latent_eps: float = 1e-6
     position: PositionSpec | None = None
     head_gate: bool = False
+    q_rank: int = 0
+    learned_sink: bool = False
+    output_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -107,7 +112,10 @@ class SinkAttentionSpec(MixerSpec):
     exp(sink_h) + sum exp(s_j), sink_h a stored number a query head, taken as it is (``scale`` does not touch it). Queries and keys are rotated
     (``position``) and then, with ``unit_norm_eps`` set, divided by their root mean square over ``head_dim`` (eps inside the
     root, no weight). ``window`` counts the keys a query sees, its own included (None: every earlier key). With ``softcap``
-    c > 0 a score s (already scaled) becomes c tanh(s / c). ``bias``: the q, k and v projections add a stored vector. The
+    c > 0 a score s (already scaled) becomes c tanh(s / c). ``bias``: the q, k and v projections add a stored vector.
+    ``keep_first`` (with a window): a query also sees the sequence's first ``keep_first`` keys. ``joined_norm_eps``: instead of rotation
+    and unit norms, all query heads side by side are divided by one root mean square and multiplied by a stored weight as wide as they
+    are, the key heads likewise. The
     cache keeps one entry [key | value] a token and key/value head, or keys and values in two planes when their sizes agree."""
     kind: str = "sink_attention"
     hidden: int = 0
@@ -123,6 +131,8 @@ class SinkAttentionSpec(MixerSpec):
     window: int | None = None
     softcap: float = 0.0
     bias: bool = False
+    keep_first: int = 0
+    joined_norm_eps: float | None = None
 
 
 @dataclass(frozen=True)
@@ -248,6 +258,23 @@ class RetentionSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class GatedLinearAttentionSpec(MixerSpec):
+    """A matrix state a head that fades by a factor a key channel and token. q = W_q h head_dim^(-1/2), k = W_k h (``num_heads`` x
+    ``head_dim``), v = W_v h (``num_heads`` x ``v_dim``); alpha = sigmoid(W_2 W_1 h + b)^(1 / ``tau``), heads x ``head_dim``, W_1 of
+    ``decay_rank`` rows; per head S <- diag(alpha) S + k v^T from S = 0, o = S^T q. Each head's o is divided by its root mean square
+    (``eps``) and multiplied by a weight of ``v_dim`` numbers that the heads share; the heads side by side are multiplied by silu(W_g h) and
+    projected out. S is kept per request in 32-bit."""
+    kind: str = "gated_linear_attention"
+    hidden: int = 0
+    num_heads: int = 0
+    head_dim: int = 0
+    v_dim: int = 0
+    tau: float = 1.0
+    decay_rank: int = 0
+    eps: float = 1e-6
+
+
+@dataclass(frozen=True)
 class SigmoidAttentionSpec(MixerSpec):
     """Grouped-query causal attention without a softmax: a visible key j gets the weight sigmoid(s_ij + b_h) of its own, and the
     weights are used as they are: nothing divides by their sum. Queries and keys are divided by their root mean square over the head (``qk_norm_eps``)
@@ -320,7 +347,8 @@ class RoutedMlpSpec(FeedForwardSpec):
     its output is multiplied. ``score`` "softmax": scores are the softmax of the logits over the experts and the
     ``identity_experts`` (router outputs beyond the experts, whose output is their input; they have no weights); with
     ``correction`` a stored vector is added to the scores for the choice only; the weights are the chosen scores times
-    ``route_scale``. ``activation``, ``limit``: as in ``GatedMlpSpec``; ``shared_limit`` is the shared expert's limit;
+    ``route_scale``. ``score`` "softmax_chosen": the largest logits are chosen and the weights are the softmax over the chosen
+    logits alone, times ``route_scale``, on the output. ``activation``, ``limit``: as in ``GatedMlpSpec``; ``shared_limit`` is the shared expert's limit;
     ``shared_gate``: the shared expert's output is multiplied by the sigmoid of one more router-like product a token."""
     kind: str = "routed_mlp"
     hidden: int = 0
@@ -430,15 +458,16 @@ class BlockSpec:
     the same two sublayers over several 32-bit residual streams, read and written through ``connection``. ``pre_norm_gated``:
     ``pre_norm_wide`` with every sublayer's output scaled by a gate of its ``connection`` (``sigmoid_gate``) before the sum.
     ``sandwich_wide``: ``pre_norm_wide`` with one more norm on every sublayer's output before it joins the stream (``mixer_out_norm``,
-    ``feed_forward_out_norm``)."""
+    ``feed_forward_out_norm``). ``post_norm_wide``: x <- x + mixer_out_norm(mixer(x)); x <- x + feed_forward_out_norm(ff(x)) over such a
+    stream: sublayers read the stream itself, rounded to the activation dtype (``input_norm`` and ``post_mixer_norm`` are None)."""
     mixer: MixerSpec
     feed_forward: FeedForwardSpec | None
-    input_norm: NormSpec
+    input_norm: NormSpec | None
     post_mixer_norm: NormSpec | None
     kind: str = "pre_norm"
     connection: ConnectionSpec | None = None
     token_input: TokenInputSpec | None = None     # ``pre_norm_wide`` only: added after the last sublayer
-    mixer_out_norm: NormSpec | None = None        # ``sandwich_wide`` only: the norms between a sublayer's output and the sum
+    mixer_out_norm: NormSpec | None = None        # ``sandwich_wide`` and ``post_norm_wide``: the norms between a sublayer's output and the sum
     feed_forward_out_norm: NormSpec | None = None
 
 

@@ -17,6 +17,11 @@
 //     that the merge kernel reduces in chunk order. The chunk size is fixed by the caller, so the order of every sum
 //     depends on the request's own length only, never on what else is in the batch.
 // Keys outside a request's visible range are never read: their shared-memory rows are zero-filled.
+//
+// keep_first > 0 (with a window): a query sees the request's first keep_first keys besides its window. The prefill kernel walks the
+// tiles of the kept keys and then the window's, leaving out the tiles between the two; a decode row's work list holds items for the
+// kept keys and for the window's keys from keep_first on. A decode item whose first key c is written as -1 - c covers its range as it
+// is, bounded by causality only: that is how the kept keys, and rows whose window has not left them yet, are listed.
 #include "tma.cuh"
 
 namespace roost {
@@ -73,13 +78,13 @@ struct Tile {
   __device__ static __forceinline__ uint32_t offset(int row, int chunk) { return (uint32_t)(row * kChunks + (chunk ^ (row & kSwizzle))) * 16u; }
 };
 
-// Loads keys [j0, j0 + ROWS) of one key/value head into a K and a V tile. Keys outside [lo, hi] are zero-filled.
+// Loads keys [j0, j0 + ROWS) of one key/value head into a K and a V tile. Keys outside [lo, hi] and not below `keep` are zero-filled.
 // A thread owns one 16-byte chunk column and every (NTHREADS / chunks)-th row. The block-table lookups of all its
 // rows are issued first, then the copies, so the lookups' latencies overlap instead of adding up in front of each copy.
 template <int D, int ROWS, int NTHREADS>
 __device__ __forceinline__ void load_kv_tile(uint32_t k_smem, uint32_t v_smem, const __nv_bfloat16* __restrict__ k_pool,
                                              const __nv_bfloat16* __restrict__ v_pool, const int32_t* __restrict__ pages,
-                                             int page_size, int page_shift, int kv_heads, int kvh, int j0, int lo, int hi, int tid) {
+                                             int page_size, int page_shift, int kv_heads, int kvh, int j0, int lo, int hi, int tid, int keep = 0) {
   constexpr int C = Tile<D>::kChunks;
   static_assert(NTHREADS % C == 0 && NTHREADS >= C, "a row's chunks must divide the threads");
   constexpr int ROWS_PER_PASS = NTHREADS / C;
@@ -90,7 +95,7 @@ __device__ __forceinline__ void load_kv_tile(uint32_t k_smem, uint32_t v_smem, c
 #pragma unroll
   for (int k = 0; k < ITER; ++k) {
     const int j = j0 + r0 + k * ROWS_PER_PASS;
-    const bool valid = j >= lo && j <= hi && (r0 + k * ROWS_PER_PASS) < ROWS;
+    const bool valid = (j >= lo || j < keep) && j <= hi && (r0 + k * ROWS_PER_PASS) < ROWS;
     page[k] = valid ? pages[page_shift >= 0 ? (j >> page_shift) : (j / page_size)] : -1;
   }
 #pragma unroll
@@ -248,7 +253,7 @@ struct RowStateM {
 template <int D, int BN, int MT>
 __device__ __forceinline__ void attend_tile_m(RowStateM<D, MT>& st, uint32_t q_smem, int q_row0, uint32_t k_smem, uint32_t v_smem,
                                               int key_row0, int j0, const int (&qpos)[MT][2], const int (&qlo)[MT][2], float scale_log2,
-                                              int lane, bool wide = false, float cap_log2 = 0.f) {
+                                              int lane, bool wide = false, float cap_log2 = 0.f, int keep = 0) {
   constexpr int NT = BN / 8;
   float s[MT][NT][4];
 #pragma unroll
@@ -303,7 +308,7 @@ __device__ __forceinline__ void attend_tile_m(RowStateM<D, MT>& st, uint32_t q_s
         for (int e = 0; e < 4; ++e) {
           const int r = e >> 1;
           const int j = j0 + n * 8 + (lane & 3) * 2 + (e & 1);
-          const float v = (j <= qpos[mt][r] && j >= qlo[mt][r]) ? s[mt][n][e] * scale_log2 : -INFINITY;
+          const float v = (j <= qpos[mt][r] && (j >= qlo[mt][r] || j < keep)) ? s[mt][n][e] * scale_log2 : -INFINITY;
           s[mt][n][e] = v;
           mx[r] = fmaxf(mx[r], v);
         }
@@ -411,7 +416,7 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
                                                                 const int32_t* __restrict__ kv_indptr,
                                                                 const int32_t* __restrict__ kv_indices, const int2* __restrict__ work,
                                                                 int q_heads, int kv_heads, int page_size, int page_shift, float scale_log2, int window,
-                                                                float cap_log2, const float* __restrict__ sinks) {
+                                                                int keep_first, float cap_log2, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // one more term, 2^(0 - m), in every row's denominator
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -458,14 +463,17 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
   const int last_row = min(row0 + BM, rows_total) - 1;
   const int hi = pos0 + last_row / group;
   const int lo = window > 0 ? max(0, pos0 + row0 / group - window + 1) : 0;
-  const int t0 = lo / BN, t1 = hi / BN;
+  const int w0 = lo / BN;                                                    // the first tile of the window
+  const int kept = min(w0, (keep_first + BN - 1) / BN);                      // tiles of kept keys in front of it
+  const int steps = kept + hi / BN - w0 + 1;
+  auto tile_at = [&](int i) { return i < kept ? i : w0 + (i - kept); };
   const int warp_first = row0 + warp * 16 * MT;
   const int warp_last = min(warp_first + 16 * MT, rows_total) - 1;
   const int warp_hi = warp_last >= warp_first ? pos0 + warp_last / group : -1;
   const int warp_lo = window > 0 ? max(0, pos0 + warp_first / group - window + 1) : 0;
 
   load_q_tile<D, BM, NT>(q_smem, q, q_start, q_heads, group, kvh, row0, rows_total, tid);
-  load_kv_tile<D, BN, NT>(k_smem[0], v_smem[0], k_pool, v_pool, pages, page_size, page_shift, kv_heads, kvh, t0 * BN, lo, hi, tid);
+  load_kv_tile<D, BN, NT>(k_smem[0], v_smem[0], k_pool, v_pool, pages, page_size, page_shift, kv_heads, kvh, tile_at(0) * BN, lo, hi, tid, keep_first);
   cp_async_commit();
 
   RowStateM<D, MT> st;
@@ -477,10 +485,10 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
     st.l[mt][0] = st.l[mt][1] = 0.f;
   }
 
-  for (int t = t0; t <= t1; ++t) {
-    const int stage = (t - t0) & 1;
-    if (t + 1 <= t1) {
-      load_kv_tile<D, BN, NT>(k_smem[stage ^ 1], v_smem[stage ^ 1], k_pool, v_pool, pages, page_size, page_shift, kv_heads, kvh, (t + 1) * BN, lo, hi, tid);
+  for (int i = 0; i < steps; ++i) {
+    const int t = tile_at(i), stage = i & 1;
+    if (i + 1 < steps) {
+      load_kv_tile<D, BN, NT>(k_smem[stage ^ 1], v_smem[stage ^ 1], k_pool, v_pool, pages, page_size, page_shift, kv_heads, kvh, tile_at(i + 1) * BN, lo, hi, tid, keep_first);
       cp_async_commit();
       cp_async_wait<1>();
     } else {
@@ -490,8 +498,8 @@ __global__ void __launch_bounds__(128) attention_prefill_kernel(const __nv_bfloa
 #pragma unroll
     for (int half = 0; half < BN / HALF; ++half) {
       const int j0 = t * BN + half * HALF;
-      if (j0 <= warp_hi && j0 + HALF - 1 >= warp_lo) {  // uniform in the warp
-        attend_tile_m<D, HALF, MT>(st, q_smem, warp * 16 * MT, k_smem[stage], v_smem[stage], half * HALF, j0, qpos, qlo, scale_log2, lane, wide, cap_log2);
+      if (j0 <= warp_hi && (j0 + HALF - 1 >= warp_lo || j0 < keep_first)) {  // uniform in the warp
+        attend_tile_m<D, HALF, MT>(st, q_smem, warp * 16 * MT, k_smem[stage], v_smem[stage], half * HALF, j0, qpos, qlo, scale_log2, lane, wide, cap_log2, keep_first);
       }
     }
     __syncthreads();
@@ -528,7 +536,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
                             const int32_t* __restrict__ kv_lens, const int32_t* __restrict__ kv_indptr,
                             const int32_t* __restrict__ kv_indices, const int4* __restrict__ work, float* __restrict__ part_o,
                             float* __restrict__ part_ml, int q_heads, int kv_heads, int page_size, int page_shift, float scale_log2, int window,
-                            int slot_limit, const float* __restrict__ sinks) {
+                            int keep_first, int slot_limit, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // added where a row's result is final, never to a partial one
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -546,7 +554,8 @@ __global__ void __launch_bounds__(NWARPS * 32)
   pdl_launch_dependents(4);
   pdl_wait(4);
   const int4 w = work[blockIdx.x];
-  const int b = w.x, kv_begin = w.y, kv_end = w.z, slot = w.w;
+  const bool windowed = w.y >= 0;     // a range written as -1 - its first key is bounded by causality only
+  const int b = w.x, kv_begin = windowed ? w.y : -1 - w.y, kv_end = w.z, slot = w.w;
   if (b < 0) return;  // padding of a fixed-size work list
   if (slot >= slot_limit) {
     if (tid == 0) atomicCAS(&g_attention_error, 0, 9);
@@ -567,7 +576,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
     const int pr = (lane >> 2) + r * 8;
     if (pr < rows_total) {
       qpos[r] = pos0 + pr / group;
-      qlo[r] = window > 0 ? max(0, qpos[r] - window + 1) : 0;
+      qlo[r] = window > 0 && windowed ? max(keep_first, qpos[r] - window + 1) : 0;
     } else {
       qpos[r] = -1;
       qlo[r] = 0;
@@ -575,7 +584,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
   }
   // keys this chunk may read: inside the chunk, not beyond the last query, not before the first query's window
   const int hi = min(kv_end - 1, kv_len - 1);
-  const int lo = max(kv_begin, window > 0 ? max(0, pos0 - window + 1) : 0);
+  const int lo = max(kv_begin, window > 0 && windowed ? max(keep_first, pos0 - window + 1) : 0);
 
   load_q_tile<D, 16, NWARPS * 32>(q_smem, q, q_start, q_heads, group, kvh, 0, rows_total, tid);
   cp_async_commit();
@@ -704,7 +713,7 @@ struct TileTma {
 };
 
 struct DecodeChunk {  // what the producer tells the consumers about a chunk
-  int b, kvh, slot, q_start, n, kv_len, lo, hi, t0, ntiles;
+  int b, kvh, slot, q_start, n, kv_len, lo, hi, t0, ntiles, windowed;
 };
 
 __device__ __forceinline__ uint32_t decode_cluster_rank() {
@@ -736,7 +745,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
                                 const int32_t* __restrict__ q_indptr, const int32_t* __restrict__ kv_lens,
                                 const int32_t* __restrict__ kv_indptr, const int32_t* __restrict__ kv_indices,
                                 const int4* __restrict__ work, int items, float* __restrict__ part_o, float* __restrict__ part_ml, int q_heads,
-                                int kv_heads, int page_size, float scale_log2, int window, int cluster_chunks, const float* __restrict__ sinks) {
+                                int kv_heads, int page_size, float scale_log2, int window, int keep_first, int cluster_chunks, const float* __restrict__ sinks) {
   const float sink = (window & ROOST_ATTENTION_SINK) ? 1.0f : 0.f;     // added where a row's result is final, never to a partial one
   const bool wide = (window & ROOST_ATTENTION_WIDE_WEIGHTS) != 0;       // the weights enter P V as two bfloat16 operands
   window &= ~(ROOST_ATTENTION_SINK | ROOST_ATTENTION_WIDE_WEIGHTS);
@@ -829,7 +838,8 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
         nc.kv_len = nkvl;
         const int pos0 = nc.kv_len - nc.n;
         nc.hi = min(nw.z - 1, nc.kv_len - 1);
-        nc.lo = max(nw.y, window > 0 ? max(0, pos0 - window + 1) : 0);
+        nc.windowed = nw.y >= 0 ? 1 : 0;     // a range written as -1 - its first key is bounded by causality only
+        nc.lo = max(nc.windowed ? nw.y : -1 - nw.y, window > 0 && nc.windowed ? max(keep_first, pos0 - window + 1) : 0);
         nc.t0 = nc.lo / TK;
         nc.ntiles = nc.hi >= nc.lo ? (nc.hi / TK - nc.t0 + 1) : 0;
         if (nc.ntiles > 0) {
@@ -988,7 +998,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
       const int pr = (lane >> 2) + r * 8;
       if (pr < rows_total) {
         qpos[r] = pos0 + pr / group;
-        qlo[r] = window > 0 ? max(0, qpos[r] - window + 1) : 0;
+        qlo[r] = window > 0 && c.windowed ? max(keep_first, qpos[r] - window + 1) : 0;
       } else {
         qpos[r] = -1;
         qlo[r] = 0;
@@ -1271,7 +1281,7 @@ constexpr int kPrefillTwoGroupsMinRows = 49152;
 template <int D, int MT>
 static int launch_prefill(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                           const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, int q_heads, int kv_heads,
-                          int page_size, float scale, int window, cudaStream_t s, float softcap = 0.f, const float* sinks = nullptr) {
+                          int page_size, float scale, int window, int keep_first, cudaStream_t s, float softcap = 0.f, const float* sinks = nullptr) {
   const size_t smem = (size_t)(64 * MT + 4 * 64) * D * 2;
   auto kernel = attention_prefill_kernel<D, MT>;
   static bool attr_set = false;  // once per process: nothing but launches happens on later calls (stream capture)
@@ -1281,7 +1291,7 @@ static int launch_prefill(const void* q, void* out, const void* k_pool, const vo
   }
   launch_kernel(kernel, dim3(items, kv_heads), dim3(128), smem, s, (const __nv_bfloat16*)q, (__nv_bfloat16*)out, (const __nv_bfloat16*)k_pool,
                 (const __nv_bfloat16*)v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, (const int2*)work, q_heads, kv_heads, page_size,
-                page_shift_of(page_size), scale * kLog2e, window, softcap * kLog2e, sinks);
+                page_shift_of(page_size), scale * kLog2e, window, keep_first, softcap * kLog2e, sinks);
   return check_launch("attention_prefill");
 }
 
@@ -1318,7 +1328,7 @@ template <int D>
 static int launch_decode_tma(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                              const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, float* part_o,
                              float* part_ml, int q_heads, int kv_heads, int page_size, long long pool_pages, float scale, int window,
-                             cudaStream_t s, int cluster_chunks, const float* sinks) {
+                             int keep_first, cudaStream_t s, int cluster_chunks, const float* sinks) {
   CUtensorMap map;
   const int box_rows = page_size < kTmaTileKeys ? page_size : kTmaTileKeys;
   const int rc = make_pool_map(&map, k_pool, v_pool, pool_pages * kv_heads * page_size, D, box_rows);
@@ -1339,7 +1349,7 @@ static int launch_decode_tma(const void* q, void* out, const void* k_pool, const
   auto kernel = box_rows == 16 ? attention_decode_tma_kernel<D, 16> : attention_decode_tma_kernel<D, 32>;
   launch_kernel_cluster(kernel, dim3(grid), dim3((kTmaConsumers + 1) * 32), smem, s, cluster_chunks > 0 ? cluster_chunks : 1, map,
                         (const __nv_bfloat16*)q, (__nv_bfloat16*)out, q_indptr, kv_lens, kv_indptr, kv_indices, (const int4*)work, items, part_o,
-                        part_ml, q_heads, kv_heads, page_size, scale * kLog2e, window, cluster_chunks, sinks);
+                        part_ml, q_heads, kv_heads, page_size, scale * kLog2e, window, keep_first, cluster_chunks, sinks);
   return check_launch("attention_decode_tma");
 }
 
@@ -1347,14 +1357,14 @@ template <int D>
 static int launch_decode(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr, const int32_t* kv_lens,
                          const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items, const int32_t* merge_work,
                          int merge_items, int merge_rows, float* part_o, float* part_ml, int q_heads, int kv_heads, int page_size,
-                         long long pool_pages, float scale, int window, cudaStream_t s, int slot_limit = kNoSlotLimit,
+                         long long pool_pages, float scale, int window, int keep_first, cudaStream_t s, int slot_limit = kNoSlotLimit,
                          const float* sinks = nullptr) {
   int rc = ROOST_OK;
   bool launched = false;
   if constexpr (D == 64 || D == 128) {
     if (slot_limit == kNoSlotLimit && decode_tma_serves(D, page_size, pool_pages, kv_heads, k_pool, v_pool)) {
       rc = launch_decode_tma<D>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, part_o, part_ml, q_heads,
-                                kv_heads, page_size, pool_pages, scale, window, s, 0, sinks);
+                                kv_heads, page_size, pool_pages, scale, window, keep_first, s, 0, sinks);
       launched = true;
     }
   }
@@ -1371,7 +1381,7 @@ static int launch_decode(const void* q, void* out, const void* k_pool, const voi
     }
     launch_kernel(kernel, dim3(items, kv_heads), dim3(NW * 32), smem, s, (const __nv_bfloat16*)q, (__nv_bfloat16*)out,
                   (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, (const int4*)work, part_o,
-                  part_ml, q_heads, kv_heads, page_size, page_shift_of(page_size), scale * kLog2e, window, slot_limit, sinks);
+                  part_ml, q_heads, kv_heads, page_size, page_shift_of(page_size), scale * kLog2e, window, keep_first, slot_limit, sinks);
     rc = check_launch("attention_decode");
   }
   if (rc != ROOST_OK || merge_items == 0) return rc;
@@ -1450,7 +1460,7 @@ extern "C" int roost_attention_mma_supported(int head_dim) {
 static int attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                              const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work, int items,
                              int tile_rows, int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                             float softcap, const float* sinks, roost_stream_t stream) {
+                             int keep_first, float softcap, const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_prefill: sizes must be positive");
   ROOST_REQUIRE(tile_rows == 64 || ((tile_rows == 128 || tile_rows == 256) && head_dim <= 128),
                 "attention_prefill: a work item has 64 packed rows, or 128 or 256 up to head size 128");
@@ -1458,34 +1468,35 @@ static int attention_prefill(const void* q, long long tokens, void* out, const v
   if (kv_heads > 65535) return fail(ROOST_ERR_UNSUPPORTED, "attention_prefill: more than 65535 key/value heads");
   if (items == 0) return ROOST_OK;
   ROOST_REQUIRE(softcap >= 0.f && (softcap == 0.f || tile_rows != 256), "attention_prefill: a cap on the scores is served by the mma.sync kernels (items of 64 or 128 packed rows)");
-  if ((tile_rows == 128 || tile_rows == 256) && tokens > 0 && !(window & ROOST_ATTENTION_WIDE_WEIGHTS) && softcap == 0.f && sinks == nullptr &&
+  if ((tile_rows == 128 || tile_rows == 256) && tokens > 0 && !(window & ROOST_ATTENTION_WIDE_WEIGHTS) && softcap == 0.f && sinks == nullptr && keep_first == 0 &&
       prefill_tc_serves(head_dim, q_heads, kv_heads, page_size, pool_pages, k_pool, v_pool, q)) {
     return launch_prefill_tc(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads,
                              head_dim, page_size, pool_pages, scale, window, (cudaStream_t)stream);
   }
-  ROOST_REQUIRE(tile_rows != 256 || (!(window & ROOST_ATTENTION_WIDE_WEIGHTS) && sinks == nullptr),
-                "attention_prefill: work items of 256 packed rows belong to the tcgen05 kernel, which takes no wide weights and no stored sinks");
+  ROOST_REQUIRE(tile_rows != 256 || (!(window & ROOST_ATTENTION_WIDE_WEIGHTS) && sinks == nullptr && keep_first == 0),
+                "attention_prefill: work items of 256 packed rows belong to the tcgen05 kernel, which takes no wide weights, stored sinks or kept keys");
+  ROOST_REQUIRE(keep_first >= 0, "attention_prefill: the number of kept keys cannot be negative");
   if (tile_rows == 128) {
     switch (head_dim) {
-      case 16: return launch_prefill<16, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
-      case 32: return launch_prefill<32, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
-      case 64: return launch_prefill<64, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
-      case 128: return launch_prefill<128, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks);
+      case 16: return launch_prefill<16, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, keep_first, (cudaStream_t)stream, softcap, sinks);
+      case 32: return launch_prefill<32, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, keep_first, (cudaStream_t)stream, softcap, sinks);
+      case 64: return launch_prefill<64, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, keep_first, (cudaStream_t)stream, softcap, sinks);
+      case 128: return launch_prefill<128, 2>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, q_heads, kv_heads, page_size, scale, window, keep_first, (cudaStream_t)stream, softcap, sinks);
       default: return fail(ROOST_ERR_UNSUPPORTED, "attention_prefill: no tensor-core kernel for this head size");
     }
   }
   ROOST_DISPATCH_HEAD_DIM(head_dim, D, return launch_prefill<D, 1>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items,
-                                                                    q_heads, kv_heads, page_size, scale, window, (cudaStream_t)stream, softcap, sinks));
+                                                                    q_heads, kv_heads, page_size, scale, window, keep_first, (cudaStream_t)stream, softcap, sinks));
   return ROOST_OK;
 }
 
 extern "C" int roost_attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool,
                                        const int32_t* q_indptr, const int32_t* kv_lens, const int32_t* kv_indptr,
                                        const int32_t* kv_indices, const int32_t* work, int items, int tile_rows, int q_heads, int kv_heads,
-                                       int head_dim, int page_size, long long pool_pages, float scale, int window, const float* sinks,
-                                       roost_stream_t stream) {
+                                       int head_dim, int page_size, long long pool_pages, float scale, int window, int keep_first,
+                                       const float* sinks, roost_stream_t stream) {
   return attention_prefill(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads, head_dim,
-                           page_size, pool_pages, scale, window, 0.f, sinks, stream);
+                           page_size, pool_pages, scale, window, keep_first, 0.f, sinks, stream);
 }
 
 // The same with a cap c on the scores: a score s (scaled) becomes c tanh(s / c) before the mask and the softmax. mma.sync kernels only.
@@ -1495,22 +1506,23 @@ extern "C" int roost_attention_prefill_capped(const void* q, long long tokens, v
                                               int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
                                               float softcap, const float* sinks, roost_stream_t stream) {
   return attention_prefill(q, tokens, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, tile_rows, q_heads, kv_heads, head_dim,
-                           page_size, pool_pages, scale, window, softcap, sinks, stream);
+                           page_size, pool_pages, scale, window, 0, softcap, sinks, stream);
 }
 
 extern "C" int roost_attention_decode(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                       const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                                       int items, const int32_t* merge_work, int merge_items, int merge_rows, float* part_o, float* part_ml,
                                       int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                                      const float* sinks, roost_stream_t stream) {
+                                      int keep_first, const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && merge_items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_decode: sizes must be positive");
   ROOST_REQUIRE(q_heads % kv_heads == 0, "attention_decode: q_heads must be a multiple of kv_heads");
   ROOST_REQUIRE(merge_items == 0 || (part_o && part_ml && merge_work), "attention_decode: the workspace for split rows is missing");
+  ROOST_REQUIRE(keep_first >= 0, "attention_decode: the number of kept keys cannot be negative");
   if (kv_heads > 65535) return fail(ROOST_ERR_UNSUPPORTED, "attention_decode: more than 65535 key/value heads");
   if (items == 0) return ROOST_OK;
   ROOST_DISPATCH_HEAD_DIM(head_dim, D, return launch_decode<D>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items,
                                                                 merge_work, merge_items, merge_rows, part_o, part_ml, q_heads, kv_heads,
-                                                                page_size, pool_pages, scale, window, (cudaStream_t)stream, kNoSlotLimit, sinks));
+                                                                page_size, pool_pages, scale, window, keep_first, (cudaStream_t)stream, kNoSlotLimit, sinks));
   return ROOST_OK;
 }
 
@@ -1533,8 +1545,8 @@ extern "C" int roost_attention_decode_cluster_supported(int head_dim, int page_s
 extern "C" int roost_attention_decode_cluster(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                               const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices,
                                               const int32_t* work, int items, int cluster_chunks, int q_heads, int kv_heads, int head_dim,
-                                              int page_size, long long pool_pages, float scale, int window, const float* sinks,
-                                              roost_stream_t stream) {
+                                              int page_size, long long pool_pages, float scale, int window, int keep_first,
+                                              const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(items >= 0 && q_heads > 0 && kv_heads > 0 && page_size > 0, "attention_decode_cluster: sizes must be positive");
   ROOST_REQUIRE(q_heads % kv_heads == 0, "attention_decode_cluster: q_heads must be a multiple of kv_heads");
   ROOST_REQUIRE(cluster_chunks == 1 || cluster_chunks == 2 || cluster_chunks == 4 || cluster_chunks == 8,
@@ -1548,10 +1560,10 @@ extern "C" int roost_attention_decode_cluster(const void* q, void* out, const vo
   const cudaStream_t s = (cudaStream_t)stream;
   if (head_dim == 64) {
     return launch_decode_tma<64>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, nullptr, nullptr, q_heads,
-                                 kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks, sinks);
+                                 kv_heads, page_size, pool_pages, scale, window, keep_first, s, cluster_chunks, sinks);
   }
   return launch_decode_tma<128>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items, nullptr, nullptr, q_heads,
-                                kv_heads, page_size, pool_pages, scale, window, s, cluster_chunks, sinks);
+                                kv_heads, page_size, pool_pages, scale, window, keep_first, s, cluster_chunks, sinks);
 }
 
 constexpr size_t kStaticScratchFloats = 4u * 1024u * 1024u;  // 16 MiB
@@ -1615,7 +1627,7 @@ extern "C" int roost_attention_decode_static(const void* q, void* out, const voi
   ROOST_DISPATCH_HEAD_DIM(head_dim, D, return launch_decode<D>(q, out, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, work, items,
                                                                 merge_work, merge_items, 16, scratch, scratch + o_padded, q_heads, kv_heads,
                                                                 page_size, /*pool_pages unknown: the cp.async kernel*/ 0, scale, window,
-                                                                (cudaStream_t)stream, /*slot_limit*/ slots));
+                                                                /*keep_first*/ 0, (cudaStream_t)stream, /*slot_limit*/ slots));
   return ROOST_OK;
 }
 

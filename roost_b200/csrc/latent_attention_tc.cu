@@ -7,7 +7,7 @@
 // denominator in 32-bit, and adds P V with V = the first `rank` numbers of the same tile; a weight enters that product as two bfloat16 operands
 // (its rounding and the remainder), so that the 32-bit weights are used to 16 bits and not to 8. The sums of a row live in registers: `NT` column tiles of 8 a warp; beyond 256 latent numbers two warps share a
 // row group, each with half of the columns and its own copy of S. A block finds its request by walking q_indptr, so the
-// kernel needs no list from the host; blocks beyond the step's tiles leave at once.
+// kernel needs no list from the host (with sinks the denominator of head h gets exp(sinks[h]) at the end); blocks beyond the step's tiles leave at once.
 #include "common.cuh"
 
 namespace roost {
@@ -44,7 +44,7 @@ __global__ void __launch_bounds__(128 * RC) latent_attention_tc_kernel(
     const __nv_bfloat16* __restrict__ q_latent, const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out,
     const __nv_bfloat16* __restrict__ pool, const int32_t* __restrict__ positions, const int32_t* __restrict__ q_indptr,
     const int32_t* __restrict__ kv_indptr, const int32_t* __restrict__ kv_indices, int tokens, int batch_rows, int heads, int nope, int rope,
-    int rank, int page_size, float scale, int window) {
+    int rank, int page_size, float scale, int window, const float* __restrict__ sinks) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int E = rank + rope;
   const int EP = ((E + 15) / 16) * 16;       // k runs in steps of 16: the columns up to EP are zero
@@ -228,6 +228,10 @@ __global__ void __launch_bounds__(128 * RC) latent_attention_tc_kernel(
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+  if (sinks != nullptr) {              // exp(sinks[h]) joins the denominator of a row that has seen its keys
+    if (m_a > -INFINITY) l_a += expf(sinks[(r0 + row_a) % heads] - m_a);
+    if (m_b > -INFINITY) l_b += expf(sinks[(r0 + row_b) % heads] - m_b);
+  }
   const float inv_a = l_a > 0.f ? 1.0f / l_a : 0.f, inv_b = l_b > 0.f ? 1.0f / l_b : 0.f;
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
@@ -255,7 +259,7 @@ extern "C" int roost_latent_attention_tc_supported(int nope, int rope, int rank)
 extern "C" int roost_latent_attention_tc(const void* q_latent, const void* q, void* out, const void* pool, const int32_t* positions,
                                          const int32_t* q_indptr, const int32_t* kv_indptr, const int32_t* kv_indices, int tokens,
                                          int batch_rows, int heads, int nope, int rope, int rank, int page_size, float scale, int window,
-                                         roost_stream_t stream) {
+                                         const float* sinks, roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && batch_rows > 0 && heads > 0 && page_size > 0, "latent_attention_tc: sizes must be positive");
   if (!roost_latent_attention_tc_supported(nope, rope, rank)) return fail(ROOST_ERR_UNSUPPORTED, "latent_attention_tc: sizes no tensor-core form serves");
   ROOST_REQUIRE((uintptr_t)q_latent % 16 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)pool % 16 == 0 && (uintptr_t)out % 4 == 0,
@@ -273,7 +277,7 @@ extern "C" int roost_latent_attention_tc(const void* q_latent, const void* q, vo
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                                            \
     launch_kernel(kernel, dim3((unsigned)blocks), dim3(128 * RC), smem, (cudaStream_t)stream, (const B*)q_latent, (const B*)q, (B*)out, \
                   (const B*)pool, positions, q_indptr, kv_indptr, kv_indices, tokens, batch_rows, heads, nope, rope, rank, page_size, scale, \
-                  window);                                                                                                            \
+                  window, sinks);                                                                                                     \
   } while (0)
   if (rank <= 64) ROOST_LA_TC(8, 1);
   else if (rank <= 128) ROOST_LA_TC(16, 1);

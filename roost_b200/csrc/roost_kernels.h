@@ -17,7 +17,7 @@
 extern "C" {
 #endif
 
-#define ROOST_ABI_VERSION 16
+#define ROOST_ABI_VERSION 17
 
 #define ROOST_OK 0
 #define ROOST_ERR_INVALID 1      /* an argument is out of range or inconsistent; nothing was launched */
@@ -115,8 +115,11 @@ int roost_paged_attention_generic(const void* q, void* out, const void* k_pool, 
  * packed row = token * group + head. With 128-row tiles, head size 64 or 128, a power-of-two number of query heads per
  * key/value head, pages of 16, 32, 64, ... rows and K and V in one allocation, prompt portions run the tcgen05 kernel
  * (attention_tc.cu) unless roost_attention_set_prefill_tc(0) was called; q then has `tokens` rows.
+ * keep_first (0 without a window): a query also sees the request's first keep_first keys, whatever its window is.
  * decode work: int32 quadruples (batch row, first key, one past the last key, partial slot or -1); rows with at most
- * 16 packed rows only; the first key of an item is a multiple of 64. merge_work: quadruples (batch row, first slot,
+ * 16 packed rows only; the first key of an item is a multiple of 64. An item whose first key c is written as -1 - c takes its range
+ * bounded by causality only; any other item takes the keys of the window from keep_first on, so a row of a model that keeps first
+ * keys lists them in an item of the first kind. merge_work: quadruples (batch row, first slot,
  * chunks | packed rows << 24, the row's first token) for rows split into several chunks; merge_rows: the most packed
  * rows any of them has.
  * part_o: float[slots * kv_heads * 16 * head_dim], part_ml: float[slots * kv_heads * 16 * 2].
@@ -133,7 +136,7 @@ void roost_attention_set_prefill_tc(int on);
 int roost_attention_prefill(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                             const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                             int items, int tile_rows, int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages,
-                            float scale, int window, const float* sinks, roost_stream_t stream);
+                            float scale, int window, int keep_first, const float* sinks, roost_stream_t stream);
 /* The same with a cap c on the scores: a scaled score s becomes c tanh(s / c) before the mask and the softmax. Served by the mma.sync
  * kernels: items of 64 or 128 packed rows (roost_attention_prefill_tile_rows_mma). */
 int roost_attention_prefill_capped(const void* q, long long tokens, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
@@ -144,7 +147,7 @@ int roost_attention_decode(const void* q, void* out, const void* k_pool, const v
                            const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                            int items, const int32_t* merge_work, int merge_items, int merge_rows, float* part_o, float* part_ml,
                            int q_heads, int kv_heads, int head_dim, int page_size, long long pool_pages, float scale, int window,
-                           const float* sinks, roost_stream_t stream);
+                           int keep_first, const float* sinks, roost_stream_t stream);
 void roost_attention_set_decode_tma(int on);
 int roost_attention_status(void);
 /* The split decode attention without partial results in memory and without a merge kernel: the grid is thread-block
@@ -159,7 +162,7 @@ int roost_attention_decode_cluster_supported(int head_dim, int page_size, long l
 int roost_attention_decode_cluster(const void* q, void* out, const void* k_pool, const void* v_pool, const int32_t* q_indptr,
                                    const int32_t* kv_lens, const int32_t* kv_indptr, const int32_t* kv_indices, const int32_t* work,
                                    int items, int cluster_chunks, int q_heads, int kv_heads, int head_dim, int page_size,
-                                   long long pool_pages, float scale, int window, const float* sinks, roost_stream_t stream);
+                                   long long pool_pages, float scale, int window, int keep_first, const float* sinks, roost_stream_t stream);
 
 /* The split decode attention without a workspace argument. It has no counterpart in the reference: it exists for
  * callers that must not allocate device memory while they run (a host that gave the whole GPU to its own arena at
@@ -283,18 +286,21 @@ int roost_gemm_simt_batched(const void* a, const void* w, void* out, int batch, 
 /* q: [tokens, heads * (nope + rope)], every head's last `rope` elements rotated in place (their first rot_dims elements,
  * pairs (i, i + rot_dims/2), angle positions[t] * inv_freq[i]). down (may be null): [tokens, rank + rope]; its first `rank`
  * elements divided by their root mean square (eps inside the root) times latent_w, its last `rope` rotated the same way, go
- * to pool[slot_mapping[t] * (rank + rope) ..] (a negative slot is skipped). */
+ * to pool[slot_mapping[t] * (rank + rope) ..] (a negative slot is skipped). interleaved: pairs (2i, 2i + 1) instead. cq (may be null):
+ * q_rank numbers a token, divided by their root mean square times cq_w into the dense cq_out. Rows of down and cq lie ld_down apart. q may
+ * be null (nothing is rotated). */
 int roost_latent_prepare(void* q, const void* down, void* pool, const float* latent_w, const double* inv_freq,
                          const int32_t* positions, const int32_t* slot_mapping, int tokens, int heads, int nope, int rope,
-                         int rot_dims, int rank, float eps, int dtype, roost_stream_t stream);
+                         int rot_dims, int rank, float eps, int interleaved, int64_t ld_down, const void* cq, void* cq_out,
+                         const float* cq_w, int q_rank, int dtype, roost_stream_t stream);
 /* q_latent: [heads, tokens, rank]; q as above (rotated); pool: [pages, page_size, rank + rope]; out: [heads, tokens, rank] =
  * sum_j p_j c_j with p the softmax over the visible keys of (q_latent . c_j + q_rot . r_j) * scale. splits > 1 deals a
  * token's key tiles to that many blocks; part: float[tokens * heads * splits * (rank + 2)]. Tables as in
  * roost_paged_attention_generic. */
 int roost_latent_attention(const void* q_latent, const void* q, void* out, float* part, const void* pool, const int32_t* positions,
                            const int32_t* token_row, const int32_t* kv_indptr, const int32_t* kv_indices, int tokens, int heads,
-                           int nope, int rope, int rank, int page_size, float scale, int window, int splits, int dtype,
-                           roost_stream_t stream);
+                           int nope, int rope, int rank, int page_size, float scale, int window, int splits, const float* sinks,
+                           int dtype, roost_stream_t stream);   /* sinks (a number a head, or null): exp(sinks[h]) joins the denominator */
 
 /* The same on the tensor cores for bfloat16 steps of many tokens (latent_attention_tc.cu): q_indptr[b] .. q_indptr[b+1] are
  * the tokens of batch row b (batch_rows rows). Serves nope and rope that are multiples of 8 and a rank that is a multiple of
@@ -303,7 +309,7 @@ int roost_latent_attention_tc_supported(int nope, int rope, int rank);
 int roost_latent_attention_tc(const void* q_latent, const void* q, void* out, const void* pool, const int32_t* positions,
                               const int32_t* q_indptr, const int32_t* kv_indptr, const int32_t* kv_indices, int tokens,
                               int batch_rows, int heads, int nope, int rope, int rank, int page_size, float scale, int window,
-                              roost_stream_t stream);
+                              const float* sinks, roost_stream_t stream);
 
 /* ---- the Mamba-2 recurrence (mamba2.cu; the layout of a state slot and the formulas are at the top of that file) ---- */
 int roost_mamba2_conv(const void* u, int64_t ld, int col, void* out, const float* w, const float* bias, const float* state,
@@ -328,7 +334,8 @@ int roost_moe_tile_rows(void);   /* rows of a tile of sorted rows */
 /* out[t, e] = x[t, :] . w[e, :] in 32-bit. */
 int roost_moe_router_logits(const void* x, const void* w, float* out, int tokens, int hidden, int experts, int dtype, roost_stream_t stream);
 /* scratch: int32[3 * tokens * top]; tiles: int32[3 * max_tiles], max_tiles >= ceil(tokens * top / tile rows) + experts;
- * counts: int32[experts], zero on entry and left at zero. mode 0: sigmoid scores, compared by logit. mode 1: softmax scores
+ * counts: int32[experts], zero on entry and left at zero. mode 2: compared by logit, the weights the softmax over the chosen logits
+ * times scale. mode 0: sigmoid scores, compared by logit. mode 1: softmax scores
  * over the `experts` routed columns of a row of `columns` logits, compared with correction[e] (may be null) added; a pair's
  * weight is score * scale. Experts from `real` on (identity experts) get sorted rows but no tiles. */
 /* wide_tiles (may be null): the same rows cut into tiles of roost_moe_wide_tile_rows() rows, int32[3 * max_wide_tiles], for
@@ -370,7 +377,26 @@ int roost_stream_step(float* streams, const void* y, const void* init_from, cons
 /* out[t, i] = act(gate[t, i], up[t, i]) over rows [gate | up] (block 0) or blocks of `block` gate then `block` up values. */
 int roost_gated_act_mul(const void* x, void* out, int tokens, int inter, int block, int act, float limit, int dtype, roost_stream_t stream);
 
+/* ---- gated linear attention (gated_linear_attention.cu): S <- diag(alpha) S + k v^T, o = S^T q a head; the slot holds S
+ * [heads, dim, vdim] ---- */
+/* alpha float[tokens, channels] = sigmoid(u[:, a_col : a_col + rank] w^T + bias)^(1 / tau); w [channels, rank] in the rows' dtype. */
+int roost_gla_prepare(const void* u, int64_t ld, int a_col, const void* w, const float* bias, float* alpha, int tokens, int channels, int rank,
+                      float tau, int dtype, roost_stream_t stream);
+/* u rows [q heads | k heads | v heads | ...], ld apart; out float[tokens, heads * vdim]. alpha as roost_gla_prepare leaves it, or null: the
+ * scan makes the decays from the rows' a1 columns itself (steps of one token a row). ws: float[roost_gla_scan_chunks(tokens, rows) * heads *
+ * dim * vdim] and ws_keep: float[chunks * heads * dim], or both null; with them rows are cut into chunks of 64 tokens that run side by side
+ * (three launches). */
+int roost_gla_scan_chunks(int tokens, int rows);
+int roost_gla_scan(const void* u, int64_t ld, float q_scale, const float* alpha, int a_col, const void* w, const float* bias, int rank, float tau,
+                   float* out, float* state, int64_t state_stride, const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads,
+                   int dim, int vdim, float* ws, float* ws_keep, int dtype, roost_stream_t stream);
+
 /* ---- attention with a sink, unit-norm heads and values of their own size (sink_attention.cu) ---- */
+/* The preparation of heads that are normed side by side: q = [all query heads] / sqrt(mean(x^2) + eps) * q_w (rows of q_out ld_q apart; it may
+ * be qkv itself), k likewise with k_w into the cache, v into the cache; nothing is rotated. */
+int roost_sink_attention_prepare_normed(const void* qkv, int64_t ld, void* q_out, int64_t ld_q, void* k_base, void* v_base, int entry,
+                                        const float* q_w, const float* k_w, const int32_t* slot_mapping, int tokens, int heads, int kv_heads,
+                                        int dim, int vdim, float eps, int page_size, int dtype, roost_stream_t stream);
 /* qkv rows [q heads | k heads | v heads] with row stride ld: rotation of interleaved pairs and unit root mean square (eps <= 0:
  * none) on q (in place, or to the dense [tokens, heads, dim] q_out when it is given) and k; k and v to the cache entry of the token's slot: ((page * kv_heads + head) * page_size + offset) *
  * entry from k_base and v_base. */
@@ -383,8 +409,9 @@ int roost_sink_attention_prepare(void* qkv, int64_t ld, void* q_out, void* k_bas
 int roost_sink_attention(const void* qkv, int64_t ld, void* out, float* part, const void* k_base, const void* v_base, int entry,
                          const int32_t* positions, const int32_t* token_row, const int32_t* kv_indptr, const int32_t* kv_indices, int tokens,
                          int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink, int splits, int tiles_per_split,
-                         int window, float softcap, const float* sinks, int dtype, roost_stream_t stream);   /* window 0: every earlier
-                                                                                                 key; softcap 0: none */
+                         int window, int keep_first, float softcap, const float* sinks, int dtype,
+                         roost_stream_t stream);   /* window 0: every earlier key; keep_first: keys from the request's first on that are seen
+                                                      whatever the window is; softcap 0: none */
 
 /* ---- the Mamba selective scan (mamba1.cu) ---- */
 /* Per (row, channel): dt = softplus(dt_raw + dt_bias); S <- exp(dt a_neg) S + dt x B; y = S . C + d_skip x; out = y silu(z). xc

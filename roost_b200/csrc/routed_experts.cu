@@ -18,6 +18,8 @@
 // products skip their rows, and combine_weighted takes the token's own row for them:
 //   combine_weighted: out[t, :] = sum_k weight[r_k] * (expert[r_k] < real ? ys[r_k, :] : x[t, :]) (+ sigmoid(gate[t]) * shared[t, :]),
 //                 r_k = inverse[t * top + k], summed in 32-bit in the order of k.
+// A third form (mode 2): the `top` largest logits are chosen as they are and a pair's weight is the softmax over the token's chosen logits
+// alone, times scale; everything else is as in mode 1.
 // The gated expert product applies the gate function of common.cuh (silu, the tanh form of GELU, the clamped swish).
 #include "common.cuh"
 
@@ -96,6 +98,7 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
     }
   }
   __syncwarp();
+  float chosen = -INFINITY;              // mode 2: lane k keeps the logit of choice k (top <= 32)
   for (int k = 0; k < top; ++k) {
     float bz = -INFINITY;
     int best = 0x7fffffff;
@@ -115,6 +118,7 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
         best = ob;
       }
     }
+    if (lane == k) chosen = bz;
     if (lane == 0) {
       z[best] = -INFINITY;               // taken
       pair_expert[(size_t)t * top + k] = best;
@@ -122,6 +126,11 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
       if (mode == 1) pair_weight[(size_t)t * top + k] = sc[best];
     }
     __syncwarp();
+  }
+  if (mode == 2) {
+    const float e = lane < top ? expf(chosen - __shfl_sync(0xffffffffu, chosen, 0)) : 0.f;     // the first choice is the largest
+    const float sum = warp_sum(e);
+    if (lane < top) pair_weight[(size_t)t * top + lane] = e / sum * scale;
   }
 }
 
@@ -177,7 +186,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const float* __restrict_
     const int dest = offs[e] + pair_rank[i];
     const float z = logits[(size_t)(i / top) * columns + e];
     token_of[dest] = i / top;
-    weight_of[dest] = mode == 1 ? pair_weight[i] : 1.0f / (1.0f + expf(-z));
+    weight_of[dest] = mode != 0 ? pair_weight[i] : 1.0f / (1.0f + expf(-z));
     expert_of[dest] = e;
     inverse[i] = dest;
   }
@@ -533,7 +542,7 @@ extern "C" int roost_moe_router_logits(const void* x, const void* w, float* out,
 // counts: int32[experts], zero on entry and left at zero (a caller keeps one buffer for all its calls on a stream).
 extern "C" int roost_moe_wide_tile_rows(void) { return kMoeWideTile; }
 
-// mode 0: sigmoid scores, compared by logit; mode 1: softmax scores over the `experts` routed columns of a row of `columns`,
+// mode 0: sigmoid scores, compared by logit; mode 2: compared by logit, the weights a softmax over the chosen logits; mode 1: softmax scores over the `experts` routed columns of a row of `columns`,
 // compared with `correction` (may be null) added, weights times `scale`. Experts from `real` on have no tiles. scratch: 3 * tokens *
 // top 32-bit words.
 extern "C" int roost_moe_route(const float* logits, int tokens, int columns, int experts, int real, int top, int mode, const float* correction,
@@ -542,7 +551,7 @@ extern "C" int roost_moe_route(const float* logits, int tokens, int columns, int
                                roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && experts > 0 && top > 0 && top <= experts && columns >= experts && real >= 0 && real <= experts,
                 "moe_route: sizes do not fit");
-  ROOST_REQUIRE(mode == 0 || mode == 1, "moe_route: the mode is 0 (sigmoid) or 1 (softmax)");
+  ROOST_REQUIRE(mode >= 0 && mode <= 2, "moe_route: the mode is 0 (sigmoid), 1 (softmax) or 2 (softmax over the chosen logits)");
   if (top > kMoeMaxTop || experts > 4096) return fail(ROOST_ERR_UNSUPPORTED, "moe_route: more than 32 choices a token or 4096 experts");
   ROOST_REQUIRE((int64_t)max_tiles >= ((int64_t)tokens * top + kMoeTile - 1) / kMoeTile + experts, "moe_route: the tile list is too short");
   ROOST_REQUIRE(counts != nullptr && scratch != nullptr, "moe_route: a pointer is null");

@@ -17,8 +17,12 @@
 //              (split z of Z takes tiles [z n, (z + 1) n), n from the step's bound on lengths); the partial sums, maxima and
 //              denominators are then combined in split order by a second kernel. A padding token (position -1) is skipped.
 //              With a window a query at position p sees the keys p - window + 1 .. p: its tiles start at the tile of the first
-//              such key, and no page before that tile's is looked up (the cache may have given it back). With a cap c a scaled
-//              score s becomes c tanh(s / c).
+//              such key, and no page before that tile's is looked up (the cache may have given it back). With keep_first the
+//              query also sees the keys 0 .. keep_first - 1: their tiles come first, the tiles between them and the window's are
+//              left out. With a cap c a scaled score s becomes c tanh(s / c).
+//   prepare_normed: the other preparation: all query heads of a token side by side are divided by one root mean square and multiplied
+//              by a weight as wide as they are, the key heads side by side likewise; nothing is rotated. Queries go to q_out (rows
+//              ld_q apart: the projection's own rows, or a dense tensor), keys and values to the token's cache slot.
 #include "common.cuh"
 
 namespace roost {
@@ -102,13 +106,76 @@ __global__ void __launch_bounds__(128) sink_prepare_kernel(T* qkv, int64_t ld, T
   }
 }
 
+// A block a token; VEC: 16-byte pieces, which never cross a head. Sums of squares in 32-bit over the projection's (rounded) outputs.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) sink_prepare_normed_kernel(const T* qkv, int64_t ld, T* q_out, int64_t ld_q, T* k_base, T* v_base, int entry,
+                                                                 const float* __restrict__ q_w, const float* __restrict__ k_w,
+                                                                 const int32_t* __restrict__ slot_mapping, int heads, int kv_heads, int dim, int vdim,
+                                                                 float eps, int page_size) {
+  __shared__ float scratch[32];
+  constexpr int N = VEC ? Vec<T>::N : 1;
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int slot = slot_mapping[t];
+  const int nq = heads * dim, nk = kv_heads * dim, nv = kv_heads * vdim;
+  const T* row = qkv + (size_t)t * ld;
+  const size_t page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
+  auto load = [&](int i, float (&v)[N]) {
+    if constexpr (VEC) {
+      Vec<T>::load(row + i, v);
+    } else {
+      v[0] = to_float(row[i]);
+    }
+  };
+  auto store = [&](T* p, const float (&v)[N]) {
+    if constexpr (VEC) {
+      Vec<T>::store(p, v);
+    } else {
+      p[0] = from_float<T>(v[0]);
+    }
+  };
+  auto mean_square = [&](int from, int n) {
+    float ss = 0.f;
+    for (int i = threadIdx.x * N; i < n; i += blockDim.x * N) {
+      float v[N];
+      load(from + i, v);
+#pragma unroll
+      for (int j = 0; j < N; ++j) ss = fmaf(v[j], v[j], ss);
+    }
+    return block_sum(ss, scratch) / (float)n;
+  };
+  pdl_wait();
+  const float inv_q = 1.0f / sqrtf(mean_square(0, nq) + eps);
+  for (int i = threadIdx.x * N; i < nq; i += blockDim.x * N) {
+    float v[N];
+    load(i, v);
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = v[j] * inv_q * q_w[i + j];
+    store(q_out + (size_t)t * ld_q + i, v);
+  }
+  if (slot < 0) return;              // a padding token: no key and no value is written
+  const float inv_k = 1.0f / sqrtf(mean_square(nq, nk) + eps);
+  for (int i = threadIdx.x * N; i < nk; i += blockDim.x * N) {
+    float v[N];
+    load(nq + i, v);
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = v[j] * inv_k * k_w[i + j];
+    store(k_base + ((page * kv_heads + i / dim) * page_size + off) * entry + i % dim, v);
+  }
+  for (int i = threadIdx.x * N; i < nv; i += blockDim.x * N) {
+    float v[N];
+    load(nq + nk + i, v);
+    store(v_base + ((page * kv_heads + i / vdim) * page_size + off) * entry + i % vdim, v);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(kSaWarps * 32) sink_attention_kernel(const T* __restrict__ qkv, int64_t ld, T* __restrict__ out, float* __restrict__ part,
                                                                      const T* __restrict__ k_base, const T* __restrict__ v_base, int entry,
                                                                      const int32_t* __restrict__ positions, const int32_t* __restrict__ token_row,
                                                                      const int32_t* __restrict__ kv_indptr, const int32_t* __restrict__ kv_indices,
                                                                      int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink,
-                                                                     int splits, int tiles_per_split, int window, float softcap,
+                                                                     int splits, int tiles_per_split, int window, int keep_first, float softcap,
                                                                      const float* __restrict__ sinks) {
   extern __shared__ float sm[];
   float* ks = sm;                                          // [tile][dim + 1]
@@ -144,16 +211,18 @@ __global__ void __launch_bounds__(kSaWarps * 32) sink_attention_kernel(const T* 
   for (int c = 0; c < kSaMaxDim / 32; ++c) acc[c] = 0.f;
   const int lo = window > 0 ? max(0, pos - window + 1) : 0;     // the first key the query sees
   const int n_tiles = pos / kSaTile + 1;
-  const int first = lo / kSaTile + z * tiles_per_split, last = min(n_tiles, first + tiles_per_split);
+  const int w0 = lo / kSaTile;                                              // the window's first tile
+  const int kept = min(w0, (keep_first + kSaTile - 1) / kSaTile);           // tiles of kept keys in front of it
+  const int first = z * tiles_per_split, last = min(kept + n_tiles - w0, first + tiles_per_split);
   const float inv_cap = softcap > 0.f ? 1.0f / softcap : 0.f;
-  for (int tile = first; tile < last; ++tile) {
-    const int k0 = tile * kSaTile;
+  for (int step = first; step < last; ++step) {
+    const int k0 = (step < kept ? step : w0 + (step - kept)) * kSaTile;
     __syncthreads();
     for (int kk = warp; kk < kSaTile; kk += kSaWarps) {      // a warp a key: its entry's address once, the lanes over its numbers
       const int kp = k0 + kk;
       float* kd = ks + (size_t)kk * (dim + 1);
       float* vd = vs + (size_t)kk * vdim;
-      if (kp <= pos && kp >= lo) {
+      if (kp <= pos && (kp >= lo || kp < keep_first)) {
         const size_t at = (((size_t)pages[kp / page_size] * kv_heads + g) * page_size + kp % page_size) * entry;
         const T* kr = k_base + at;
         const T* vr = v_base + at;
@@ -183,7 +252,7 @@ __global__ void __launch_bounds__(kSaWarps * 32) sink_attention_kernel(const T* 
     }
     s *= scale;
     if (softcap > 0.f) s = softcap * tanhf(s * inv_cap);
-    if (k0 + lane > pos || k0 + lane < lo) s = -INFINITY;
+    if (k0 + lane > pos || (k0 + lane < lo && k0 + lane >= keep_first)) s = -INFINITY;
     const float m_new = fmaxf(m, warp_max(s));
     const float p = s > -INFINITY ? expf(s - m_new) : 0.f;
     const float keep = m > -INFINITY ? expf(m - m_new) : 0.f;
@@ -284,13 +353,34 @@ extern "C" int roost_sink_attention_prepare(void* qkv, int64_t ld, void* q_out, 
   return check_launch("sink_attention_prepare");
 }
 
+extern "C" int roost_sink_attention_prepare_normed(const void* qkv, int64_t ld, void* q_out, int64_t ld_q, void* k_base, void* v_base, int entry,
+                                                   const float* q_w, const float* k_w, const int32_t* slot_mapping, int tokens, int heads, int kv_heads,
+                                                   int dim, int vdim, float eps, int page_size, int dtype, roost_stream_t stream) {
+  ROOST_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0 && eps > 0.f,
+                "sink_attention_prepare_normed: sizes and eps must be positive");
+  ROOST_REQUIRE(qkv && q_out && k_base && v_base && q_w && k_w && slot_mapping, "sink_attention_prepare_normed: a pointer is null");
+  ROOST_REQUIRE(ld >= (int64_t)(heads + kv_heads) * dim + (int64_t)kv_heads * vdim && ld_q >= (int64_t)heads * dim && entry >= dim && entry >= vdim,
+                "sink_attention_prepare_normed: a row or a cache entry is too narrow");
+  if (tokens == 0) return ROOST_OK;
+  const int n = dtype == ROOST_F32 ? 4 : 8;
+  const bool vec = dim % n == 0 && vdim % n == 0 && entry % n == 0 && ld % n == 0 && ld_q % n == 0 &&
+                   ((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_base | (uintptr_t)v_base) % 16 == 0;
+  const int threads = heads * dim >= 1024 ? 256 : 128;
+  ROOST_DISPATCH_DTYPE(dtype, T, {
+    auto kernel = vec ? sink_prepare_normed_kernel<T, true> : sink_prepare_normed_kernel<T, false>;
+    launch_kernel(kernel, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, (const T*)qkv, ld, (T*)q_out, ld_q, (T*)k_base, (T*)v_base, entry, q_w,
+                  k_w, slot_mapping, heads, kv_heads, dim, vdim, eps, page_size);
+  });
+  return check_launch("sink_attention_prepare_normed");
+}
+
 extern "C" int roost_sink_attention(const void* qkv, int64_t ld, void* out, float* part, const void* k_base, const void* v_base, int entry,
                                     const int32_t* positions, const int32_t* token_row, const int32_t* kv_indptr, const int32_t* kv_indices,
                                     int tokens, int heads, int kv_heads, int dim, int vdim, int page_size, float scale, int sink, int splits,
-                                    int tiles_per_split, int window, float softcap, const float* sinks, int dtype, roost_stream_t stream) {
+                                    int tiles_per_split, int window, int keep_first, float softcap, const float* sinks, int dtype, roost_stream_t stream) {
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && kv_heads > 0 && dim > 0 && vdim > 0 && page_size > 0, "sink_attention: sizes must be positive");
   ROOST_REQUIRE(heads % kv_heads == 0, "sink_attention: the query heads are no multiple of the key/value heads");
-  ROOST_REQUIRE(window >= 0 && softcap >= 0.f, "sink_attention: the window and the scores' cap cannot be negative");
+  ROOST_REQUIRE(window >= 0 && keep_first >= 0 && softcap >= 0.f, "sink_attention: the window, the kept keys and the scores' cap cannot be negative");
   ROOST_REQUIRE(splits >= 1 && tiles_per_split >= 1 && (splits == 1 || part != nullptr), "sink_attention: splits need a workspace for their partials");
   if (dim > kSaMaxDim || vdim > kSaMaxDim) return fail(ROOST_ERR_UNSUPPORTED, "sink_attention: heads or values beyond 512 numbers");
   const int group = heads / kv_heads;
@@ -304,7 +394,7 @@ extern "C" int roost_sink_attention(const void* qkv, int64_t ld, void* out, floa
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_kernel(kernel, grid, dim3(kSaWarps * 32), smem, (cudaStream_t)stream, (const T*)qkv, ld, (T*)out, splits > 1 ? part : (float*)nullptr,
                   (const T*)k_base, (const T*)v_base, entry, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, page_size,
-                  scale, sink, splits, tiles_per_split, window, softcap, sinks);
+                  scale, sink, splits, tiles_per_split, window, keep_first, softcap, sinks);
     if (splits > 1)
       launch_kernel(sink_merge_kernel<T>, dim3(tokens, heads), dim3(128), 0, (cudaStream_t)stream, (const float*)part, (T*)out, positions, heads,
                     vdim, splits);

@@ -94,7 +94,7 @@ __global__ void wide_rms_norm_kernel(float* stream, const T* __restrict__ addend
 
 // The norm after a sublayer and the norm before the next one in one pass over a 32-bit stream. One block per output row: the addend's
 // root mean square, s = stream + addend * inv * post_w (written back unless the rows are gathered), then s's root mean square and the
-// output, rounded once. Rows a block covers with eight numbers a thread stay in registers (VEC); others go through shared memory.
+// output, rounded once. Without w the output is s itself, rounded once (a next sublayer that reads the stream as it is). Rows a block covers with eight numbers a thread stay in registers (VEC); others go through shared memory.
 template <typename T, bool VEC>
 __global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend, const float* __restrict__ post_w, float post_eps,
                                      const float* __restrict__ w, T* __restrict__ out, const int32_t* __restrict__ rows, int hidden, float eps) {
@@ -116,7 +116,7 @@ __global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend
 #pragma unroll
       for (int j = 0; j < 8; j += 4) {
         *reinterpret_cast<float4*>(pw + j) = *reinterpret_cast<const float4*>(post_w + i8 + j);
-        *reinterpret_cast<float4*>(nw + j) = *reinterpret_cast<const float4*>(w + i8 + j);
+        if (w != nullptr) *reinterpret_cast<float4*>(nw + j) = *reinterpret_cast<const float4*>(w + i8 + j);
       }
     }
     pdl_wait();
@@ -141,15 +141,17 @@ __global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend
       s[j] = s[j] + a[j] * inv_a * pw[j];
       ss = fmaf(s[j], s[j], ss);
     }
-    ss = block_sum(ss, scratch);
+    if (w != nullptr) ss = block_sum(ss, scratch);
     if (!live) return;
     if (!rows) {
       *reinterpret_cast<float4*>(s_row + i8) = make_float4(s[0], s[1], s[2], s[3]);
       *reinterpret_cast<float4*>(s_row + i8 + 4) = make_float4(s[4], s[5], s[6], s[7]);
     }
-    const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
+    if (w != nullptr) {
+      const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s[j] = s[j] * inv * nw[j];
+      for (int j = 0; j < 8; ++j) s[j] = s[j] * inv * nw[j];
+    }
     if constexpr (sizeof(T) == 2) {
       Vec<T>::store(o_row + i8, s);
     } else {
@@ -173,7 +175,9 @@ __global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend
       if (!rows) s_row[i] = s;
       keep[i] = s;
       ss = fmaf(s, s, ss);
+      if (w == nullptr) o_row[i] = from_float<T>(s);
     }
+    if (w == nullptr) return;
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)hidden + eps);
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) o_row[i] = from_float<T>(keep[i] * inv * w[i]);
@@ -419,7 +423,7 @@ extern "C" int roost_sandwich_norm(float* stream, const void* addend, const floa
                                    const int32_t* rows, int n_out, int hidden, float eps, int dtype, roost_stream_t stream_handle) {
   ROOST_REQUIRE(n_out >= 0 && hidden > 0, "sandwich_norm: rows and hidden must be positive");
   ROOST_REQUIRE(eps > 0.f && post_eps > 0.f, "sandwich_norm: both eps must be positive");
-  ROOST_REQUIRE(stream && addend && post_w && w && out, "sandwich_norm: a pointer is null");
+  ROOST_REQUIRE(stream && addend && post_w && out, "sandwich_norm: a pointer is null");
   if (n_out == 0) return ROOST_OK;
   const bool vec = hidden % 8 == 0 && hidden <= 8192 &&
                    (((uintptr_t)stream | (uintptr_t)addend | (uintptr_t)post_w | (uintptr_t)w | (uintptr_t)out) % 16 == 0);

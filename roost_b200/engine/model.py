@@ -159,10 +159,14 @@ class Model:
 
 
 def read_model_config(model_dir):
-    """(architecture entry, typed configuration, reader) of a model folder."""
+    """(architecture entry, typed configuration, reader) of a model folder. A configuration with sizes that only the checkpoint's tensors
+    give (``take_shapes``) gets their shapes."""
     reader = ConfigReader.from_path(Path(model_dir))
     arch = registry.resolve(reader)
-    return arch, arch.read_config(reader), reader
+    cfg = arch.read_config(reader)
+    if hasattr(cfg, "take_shapes"):
+        cfg.take_shapes(weight_loader.checkpoint_shapes(model_dir))
+    return arch, cfg, reader
 
 
 def load_model(model_dir, dtype: torch.dtype, device="cuda", kernels=None) -> Model:

@@ -14,7 +14,7 @@ import torch
 
 from . import build
 
-ABI_VERSION = 16
+ABI_VERSION = 17
 F32, BF16 = 0, 1
 GATE_FUNCTIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}   # the codes of csrc/roost_kernels.h
 
@@ -84,14 +84,14 @@ _SIGNATURES = {
     "roost_attention_set_prefill_tc": [c_int],
     "roost_attention_prefill_tile_rows_mma": [c_int, c_int, ctypes.c_longlong],
     "roost_attention_prefill": [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p, c_void_p],
+                                c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_int, c_void_p, c_void_p],
     "roost_attention_prefill_capped": [c_void_p, ctypes.c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                        c_int, c_int, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_float, c_void_p, c_void_p],
     "roost_attention_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int,
-                               c_void_p, c_void_p],
+                               c_int, c_void_p, c_void_p],
     "roost_attention_decode_cluster": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                                       c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_void_p, c_void_p],
+                                       c_int, c_int, c_int, c_int, ctypes.c_longlong, c_float, c_int, c_int, c_void_p, c_void_p],
     "roost_attention_decode_cluster_supported": [c_int, c_int, ctypes.c_longlong, c_int, c_void_p, c_void_p],
     "roost_sample_penalise": [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_void_p],
@@ -123,12 +123,18 @@ _SIGNATURES = {
     "roost_gemm_simt_batched": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int64, c_int64, c_int64,
                                 c_int, c_int, c_void_p],
     "roost_latent_prepare": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_float, c_int, c_void_p],
+                             c_float, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "roost_latent_attention": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                               c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+                               c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_void_p],
     "roost_latent_attention_tc_supported": [c_int, c_int, c_int],
     "roost_latent_attention_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                                  c_int, c_int, c_int, c_float, c_int, c_void_p],
+                                  c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
+    "roost_gla_prepare": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    "roost_gla_scan_chunks": [c_int, c_int],
+    "roost_gla_scan": [c_void_p, c_int64, c_float, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int64, c_void_p, c_void_p,
+                       c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
+    "roost_sink_attention_prepare_normed": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                            c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
     "roost_mamba2_conv": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_int,
                           c_int, c_int, c_int, c_int, c_void_p],
     "roost_mamba2_conv_state": [c_void_p, c_int64, c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -153,7 +159,7 @@ _SIGNATURES = {
     "roost_sink_attention_prepare": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                      c_int, c_float, c_int, c_int, c_float, c_int, c_void_p],
     "roost_sink_attention": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
+                             c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "roost_wide_rms_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "roost_normed_mean": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "roost_pair_embedding": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
@@ -294,19 +300,21 @@ class KernelLibrary:
             return 0
         return size if self._lib.roost_attention_decode_cluster_supported(d, page, pages, nkv, _ptr(k_pool), _ptr(v_pool)) else 0
 
-    def decode_split_for(self, rows: int, kv_cap: int, k_pool: torch.Tensor, v_pool: torch.Tensor) -> tuple[int, int]:
+    def decode_split_for(self, rows: int, kv_cap: int, k_pool: torch.Tensor, v_pool: torch.Tensor, chunks_of=None) -> tuple[int, int]:
         """(keys per work item, CTAs a cluster or 0) of the split decode attention for a step of ``rows`` rows whose
         requests hold at most ``kv_cap`` keys (the bounds of the captured step, so that every replay of it agrees). Where
         clusters serve, the smallest chunk of 128, 256, 512 or 1024 keys whose clusters all run at once: more CTAs pull
         on the memory and the merge costs no kernel (one row of 1,024 keys: 7.7 us in chunks of 128, 12.6 us in chunks of
         512). Else the chunk of ``decode_chunk_for`` through the merge kernel. A row's bits depend on the chunk, so on
-        the step's size class, within rounding."""
+        the step's size class, within rounding. ``chunks_of`` (chunk -> the most work items a row has): for rows that
+        are not listed as one range of keys."""
+        reach = (lambda chunk: chunks_of(chunk) * chunk) if chunks_of is not None else (lambda chunk: kv_cap)
         if self.decode_cluster and kv_cap > 0:
             for chunk in (128, 256, 512, 1024):
-                cluster = self.decode_cluster_for(rows, kv_cap, chunk, k_pool, v_pool)
+                cluster = self.decode_cluster_for(rows, reach(chunk), chunk, k_pool, v_pool)
                 if cluster:
                     return chunk, cluster
-        return self.decode_chunk_for(rows, kv_cap, k_pool.shape[1]), 0
+        return self.decode_chunk_for(rows, reach(self.decode_chunk), k_pool.shape[1]), 0
 
     # ------------------------------------------------------------------ ops
     def embedding(self, table: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
@@ -438,14 +446,15 @@ class KernelLibrary:
 
     def attention_mma(self, q, k_pool, v_pool, q_indptr, kv_lens, kv_indptr, kv_indices, plan, scale: float,
                       window: int | None, sink: bool = False, wide_weights: bool = False, softcap: float = 0.0,
-                      sinks: torch.Tensor | None = None) -> torch.Tensor:
+                      sinks: torch.Tensor | None = None, keep_first: int = 0) -> torch.Tensor:
         """Tensor-core attention (bfloat16). ``plan``: an ``AttentionPlan`` whose work lists are on the device. ``sink``: one is
         added to the softmax's denominator (a key of score 0 that has no value), or exp(sinks[h]) of head h with ``sinks`` (float32, one a
         query head). ``wide_weights``: the softmax weights enter P V as two
         bfloat16 operands (16 bits of the 32-bit weights); the plan's prefill items must then come from
         ``attention_prefill_tile_rows(..., tensor_memory=False)``. ``softcap`` c > 0: a scaled score s becomes c tanh(s / c); the
         prompt kernels on mma.sync serve it (items from ``tensor_memory=False``), the decode kernels do not: the plan must hold no
-        decode items then."""
+        decode items then. ``keep_first``: with a window, a query also sees its request's first ``keep_first`` keys; the plan's decode
+        items must list them (``attention_work(..., keep_first=)``)."""
         _need(q, "q", torch.bfloat16); _need(k_pool, "k_pool", torch.bfloat16); _need(v_pool, "v_pool", torch.bfloat16)
         T, nq, d = q.shape
         _, nkv, page, d2 = k_pool.shape
@@ -457,6 +466,8 @@ class KernelLibrary:
             _need(sinks, "sinks", torch.float32)
             if not sink or sinks.numel() != nq:
                 raise KernelError("attention_mma: stored sinks come with ``sink`` and are one number a query head")
+        if keep_first and (not window or softcap):
+            raise KernelError("attention_mma: kept keys come with a window and without a cap on the scores")
         if softcap and plan.decode_items:
             raise KernelError("attention_mma: the decode kernels know no cap on the scores")
         if plan.prefill_items and softcap:
@@ -466,11 +477,11 @@ class KernelLibrary:
         elif plan.prefill_items:
             self._call("roost_attention_prefill", _ptr(q), T, _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.prefill_work), plan.prefill_items, plan.prefill_tile_rows, nq, nkv, d, page,
-                       k_pool.shape[0], scale, w, _ptr(sinks), _stream())
+                       k_pool.shape[0], scale, w, int(keep_first), _ptr(sinks), _stream())
         if plan.decode_items and plan.cluster_chunks:
             self._call("roost_attention_decode_cluster", _ptr(q), _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.decode_work), plan.decode_items, plan.cluster_chunks, nq, nkv, d, page,
-                       k_pool.shape[0], scale, w, _ptr(sinks), _stream())
+                       k_pool.shape[0], scale, w, int(keep_first), _ptr(sinks), _stream())
         elif plan.decode_items:
             part_o = part_ml = None
             if plan.slots:
@@ -478,8 +489,8 @@ class KernelLibrary:
                 part_ml = torch.empty((plan.slots * nkv * 16 * 2,), dtype=torch.float32, device=q.device)
             self._call("roost_attention_decode", _ptr(q), _ptr(out), _ptr(k_pool), _ptr(v_pool), _ptr(q_indptr), _ptr(kv_lens),
                        _ptr(kv_indptr), _ptr(kv_indices), _ptr(plan.decode_work), plan.decode_items, _ptr(plan.merge_work),
-                       plan.merge_items, plan.merge_rows, _ptr(part_o), _ptr(part_ml), nq, nkv, d, page, k_pool.shape[0], scale, w, _ptr(sinks), _stream(),
-                       launches=2 if plan.merge_items else 1)
+                       plan.merge_items, plan.merge_rows, _ptr(part_o), _ptr(part_ml), nq, nkv, d, page, k_pool.shape[0], scale, w, int(keep_first), _ptr(sinks),
+                       _stream(), launches=2 if plan.merge_items else 1)
         return out
 
     def gemm_simt(self, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:
@@ -648,21 +659,39 @@ class KernelLibrary:
         return out
 
     # ------------------------------------------------------------------ latent attention
-    def latent_prepare(self, q, down, pool, latent_w, inv_freq, rotary_dim, positions, slot_mapping, heads, nope, rope, rank, eps, page_size) -> None:
-        """Rotates the heads' rotated query parts in place and, when ``down`` is given, writes the tokens' cache entries."""
-        _need(q, "q"); _need(positions, "positions", torch.int32)
+    def latent_prepare(self, q, down, pool, latent_w, inv_freq, rotary_dim, positions, slot_mapping, heads, nope, rope, rank, eps, page_size, interleaved: bool = False,
+                       cq: torch.Tensor | None = None, cq_w: torch.Tensor | None = None) -> torch.Tensor | None:
+        """Rotates the heads' rotated query parts in place (``q`` None: nothing is rotated) and, when ``down`` is given, writes the tokens'
+        cache entries. ``interleaved``: element 2i of a rotated part is paired with 2i + 1. ``cq`` (a latent the queries are made from later): its
+        norm under ``cq_w`` is returned, dense. ``down`` and ``cq`` may be ranges of the columns of wider rows."""
+        _need(positions, "positions", torch.int32)
+        lead = q if q is not None else (cq if cq is not None else down)
+        if lead is None:
+            raise KernelError("latent_prepare: neither queries nor a latent are given")
+        if q is not None:
+            _need(q, "q")
         if rotary_dim:
             _need(inv_freq, "inv_freq", torch.float64)
-        T = q.shape[0]
-        if q.shape[1] != heads * (nope + rope) or (rotary_dim and inv_freq.numel() != rotary_dim // 2):
+        T, dtype = lead.shape[0], lead.dtype
+        if (q is not None and q.shape[1] != heads * (nope + rope)) or (rotary_dim and inv_freq.numel() != rotary_dim // 2):
             raise KernelError("latent_prepare: q or inv_freq do not fit the sizes")
+        cq_out = None
+        if cq is not None:
+            _need_rows(cq, "cq"); _need(cq_w, "cq_w", torch.float32)
+            if cq_w.numel() != cq.shape[1]:
+                raise KernelError("latent_prepare: the queries' latent and its weight differ in size")
+            cq_out = torch.empty(cq.shape, dtype=dtype, device=cq.device)
+        if down is not None and cq is not None and T > 1 and down.stride(0) != cq.stride(0):
+            raise KernelError("latent_prepare: the two latents must be columns of the same rows")
         if down is not None:
-            _need(down, "down", q.dtype); _need(pool, "pool", q.dtype); _need(latent_w, "latent_w", torch.float32)
+            _need_rows(down, "down", dtype); _need(pool, "pool", dtype); _need(latent_w, "latent_w", torch.float32)
             _need(slot_mapping, "slot_mapping", torch.int32)
             if tuple(down.shape) != (T, rank + rope) or tuple(pool.shape[1:]) != (1, page_size, rank + rope) or latent_w.numel() != rank:
                 raise KernelError("latent_prepare: down, pool or the latent's weight do not fit the sizes")
+        ld_down = down.stride(0) if down is not None else (cq.stride(0) if cq is not None else 0)
         self._call("roost_latent_prepare", _ptr(q), _ptr(down), _ptr(pool), _ptr(latent_w), _ptr(inv_freq) if rotary_dim else None, _ptr(positions), _ptr(slot_mapping),
-                   T, heads, nope, rope, rotary_dim, rank, eps, dtype_code(q.dtype), _stream())
+                   T, heads, nope, rope, rotary_dim, rank, eps, 1 if interleaved else 0, ld_down, _ptr(cq), _ptr(cq_out), _ptr(cq_w), cq.shape[1] if cq is not None else 0, dtype_code(dtype), _stream())
+        return cq_out
 
     def latent_splits_for(self, tokens: int, heads: int, window: int | None, kv_cap: int) -> int:
         """Blocks a token's keys are dealt to: 1 when the step's (token, 8 heads) blocks fill the device by themselves, else as
@@ -678,10 +707,16 @@ class KernelLibrary:
     LATENT_TC_MIN_ROWS = 128    # packed (token, head) rows from which a bfloat16 step runs the tensor-core form
 
     def latent_attention(self, q_latent, q, pool, positions, token_row, kv_indptr, kv_indices, heads, nope, rope, rank, scale, window,
-                         kv_cap: int = 0, few_rows: bool = False, q_indptr: torch.Tensor | None = None) -> torch.Tensor:
+                         kv_cap: int = 0, few_rows: bool = False, q_indptr: torch.Tensor | None = None,
+                         sinks: torch.Tensor | None = None) -> torch.Tensor:
         """Attention in the latent space: out [heads, tokens, rank]. bfloat16 steps of many tokens (prompt portions) run on
         the tensor cores where the sizes allow; steps of few rows (decode) and float32 run the 32-bit form, a token's keys
-        dealt to several blocks when the step alone would not fill the device."""
+        dealt to several blocks when the step alone would not fill the device. ``sinks`` (float32, one a head): exp(sinks[h]) joins the
+        softmax's denominator."""
+        if sinks is not None:
+            _need(sinks, "sinks", torch.float32)
+            if sinks.numel() != heads:
+                raise KernelError("latent_attention: stored sinks are one number a head")
         _need(q_latent, "q_latent"); _need(q, "q", q_latent.dtype); _need(pool, "pool", q.dtype)
         for n, t in (("positions", positions), ("token_row", token_row), ("kv_indptr", kv_indptr), ("kv_indices", kv_indices)):
             _need(t, n, torch.int32)
@@ -694,13 +729,13 @@ class KernelLibrary:
             _need(q_indptr, "q_indptr", torch.int32)
             self._call("roost_latent_attention_tc", _ptr(q_latent), _ptr(q), _ptr(out), _ptr(pool), _ptr(positions), _ptr(q_indptr),
                        _ptr(kv_indptr), _ptr(kv_indices), T, q_indptr.numel() - 1, heads, nope, rope, rank, pool.shape[2], scale,
-                       int(window) if window else 0, _stream())
+                       int(window) if window else 0, _ptr(sinks), _stream())
             return out
         splits = self.latent_splits_for(T, heads, window, kv_cap) if kv_cap else 1
         part = torch.empty((T * heads * splits * (rank + 2),), dtype=torch.float32, device=q.device) if splits > 1 else None
         self._call("roost_latent_attention", _ptr(q_latent), _ptr(q), _ptr(out), _ptr(part), _ptr(pool), _ptr(positions), _ptr(token_row),
                    _ptr(kv_indptr), _ptr(kv_indices), T, heads, nope, rope, rank, pool.shape[2], scale, int(window) if window else 0, splits,
-                   dtype_code(q.dtype), _stream(), launches=2 if splits > 1 else 1)
+                   _ptr(sinks), dtype_code(q.dtype), _stream(), launches=2 if splits > 1 else 1)
         return out
 
     # ------------------------------------------------------------------ prompt portions over keys and values carried out of a latent cache
@@ -792,15 +827,19 @@ class KernelLibrary:
                   routed: int | None = None, real: int | None = None) -> MoeRoute:
         """``score`` "sigmoid": the weights are the sigmoid of the chosen logits. "softmax": scores are the softmax over the first
         ``routed`` columns (default all), ``correction`` is added for the choice only, the weights are score * ``scale``; experts
-        from ``real`` on are identity experts (sorted rows, no tiles)."""
+        from ``real`` on are identity experts (sorted rows, no tiles). "softmax_chosen": the largest logits are chosen and the weights are the
+        softmax over the chosen logits alone, times ``scale``."""
         _need(logits, "logits", torch.float32)
         T, columns = logits.shape
         E = columns if routed is None else routed
         real = E if real is None else real
-        if score not in ("sigmoid", "softmax"):
-            raise KernelError(f"moe_route: score '{score}' is neither sigmoid nor softmax")
+        modes = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
+        if score not in modes:
+            raise KernelError(f"moe_route: score '{score}' is none of {', '.join(modes)}")
         if correction is not None:
             _need(correction, "correction", torch.float32)
+            if score != "softmax":
+                raise KernelError("moe_route: a correction belongs to softmax scores")
             if correction.numel() != E:
                 raise KernelError("moe_route: the correction does not have one number a routed expert")
         counts = getattr(self, "_moe_counts", None)
@@ -821,7 +860,7 @@ class KernelLibrary:
         wide_tiles, at = (ints[at : at + 3 * max_wide] if max_wide else None), at + 3 * max_wide
         scratch = ints[at : at + 3 * rows]
         weight = torch.empty((rows,), dtype=torch.float32, device=dev)
-        self._call("roost_moe_route", _ptr(logits), T, columns, E, real, top, 1 if score == "softmax" else 0, _ptr(correction), float(scale),
+        self._call("roost_moe_route", _ptr(logits), T, columns, E, real, top, modes[score], _ptr(correction), float(scale),
                    _ptr(token), _ptr(weight), _ptr(expert), _ptr(inverse), _ptr(offsets), _ptr(tiles), max_tiles, _ptr(wide_tiles), max_wide,
                    _ptr(scratch), _ptr(counts), _stream(), launches=2)
         return MoeRoute(top=top, rows=rows, token=token, weight=weight, expert=expert, inverse=inverse, offsets=offsets, tiles=tiles,
@@ -969,6 +1008,27 @@ class KernelLibrary:
                    _ptr(slot_mapping), qkv.shape[0], heads, kv_heads, dim, vdim, rotary_dim, float(eps) if eps else 0.0, page_size,
                    1 if halves else 0, float(amplitude), dtype_code(qkv.dtype), _stream())
 
+    def sink_attention_prepare_normed(self, qkv, k_pool, v_pool, slot_mapping, heads, kv_heads, dim, vdim, q_w, k_w, eps, page_size,
+                                      q_out: torch.Tensor | None = None) -> None:
+        """Instead of ``sink_attention_prepare``: all query heads of a token side by side are divided by one root mean square and multiplied by
+        ``q_w`` (as wide as they are), the key heads likewise with ``k_w``; nothing is rotated."""
+        if q_out is not None:
+            _need(q_out, "q_out", qkv.dtype)
+            if tuple(q_out.shape) != (qkv.shape[0], heads, dim):
+                raise KernelError("sink_attention_prepare_normed: q_out is not [tokens, heads, dim]")
+        _need_rows(qkv, "qkv"); _need(k_pool, "k_pool", qkv.dtype); _need(slot_mapping, "slot_mapping", torch.int32)
+        _need(q_w, "q_w", torch.float32); _need(k_w, "k_w", torch.float32)
+        if v_pool is not None:
+            _need(v_pool, "v_pool", qkv.dtype)
+        if qkv.shape[1] < (heads + kv_heads) * dim + kv_heads * vdim or k_pool.shape[1] != kv_heads or k_pool.shape[2] != page_size:
+            raise KernelError("sink_attention_prepare_normed: qkv or the pool do not fit the sizes")
+        if q_w.numel() != heads * dim or k_w.numel() != kv_heads * dim:
+            raise KernelError("sink_attention_prepare_normed: a weight is as wide as the heads side by side")
+        kb, vb, entry = self._sink_cache(k_pool, v_pool, dim, vdim)
+        q_dst, ld_q = (qkv, qkv.stride(0)) if q_out is None else (q_out, heads * dim)
+        self._call("roost_sink_attention_prepare_normed", _ptr(qkv), qkv.stride(0), _ptr(q_dst), ld_q, kb, vb, entry, _ptr(q_w), _ptr(k_w),
+                   _ptr(slot_mapping), qkv.shape[0], heads, kv_heads, dim, vdim, float(eps), page_size, dtype_code(qkv.dtype), _stream())
+
     def sink_splits_for(self, tokens: int, gy: int, kv_cap: int) -> tuple[int, int]:
         """(blocks a token's key tiles are dealt to, tiles a block): 1 when the step's blocks fill the device by themselves,
         else as many as give two blocks an SM, up to 32 and to the tiles the bound on the requests' lengths allows, so that
@@ -981,10 +1041,14 @@ class KernelLibrary:
         return -(-tiles // per), per
 
     def sink_attention(self, qkv, k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, scale, sink,
-                       kv_cap: int = 0, window: int | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None) -> torch.Tensor:
+                       kv_cap: int = 0, window: int | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None,
+                       keep_first: int = 0) -> torch.Tensor:
         """Attention of the step's (prepared) queries over the paged cache in 32-bit arithmetic: out [T, heads * vdim]. ``window``:
         the keys a query sees, its own included (None: all); ``softcap`` c > 0: a scaled score s becomes c tanh(s / c); ``sinks`` (float32, one
-        a query head): exp(sinks[h]) is the sink's term in the denominator instead of one."""
+        a query head): exp(sinks[h]) is the sink's term in the denominator instead of one. ``keep_first`` (with a window): the request's first
+        ``keep_first`` keys are seen whatever the window is."""
+        if keep_first and not window:
+            raise KernelError("sink_attention: kept keys come with a window")
         _need(qkv, "qkv"); _need(k_pool, "k_pool", qkv.dtype)
         for n, t in (("positions", positions), ("token_row", token_row), ("kv_indptr", kv_indptr), ("kv_indices", kv_indices)):
             _need(t, n, torch.int32)
@@ -997,12 +1061,13 @@ class KernelLibrary:
         out = torch.empty((T, heads * vdim), dtype=qkv.dtype, device=qkv.device)
         gy = kv_heads * (-(-(heads // kv_heads) // 8))
         # a window's keys span at most window + 31 positions' worth of tiles, whatever the requests' lengths are
-        span = min(kv_cap, window + 62) if (window and kv_cap) else kv_cap
+        # (and those of the kept keys keep_first + 31 more)
+        span = min(kv_cap, window + 62 + (keep_first + 31 if keep_first else 0)) if (window and kv_cap) else kv_cap
         splits, per = self.sink_splits_for(T, gy, span) if span else (1, 1 << 24)
         part = torch.empty((T * heads * splits * (vdim + 2),), dtype=torch.float32, device=qkv.device) if splits > 1 else None
         self._call("roost_sink_attention", _ptr(qkv), qkv.stride(0), _ptr(out), _ptr(part), kb, vb, entry, _ptr(positions), _ptr(token_row),
                    _ptr(kv_indptr), _ptr(kv_indices), T, heads, kv_heads, dim, vdim, k_pool.shape[2], float(scale), 1 if sink else 0, splits, per,
-                   int(window or 0), float(softcap or 0.0), _ptr(sinks), dtype_code(qkv.dtype), _stream(), launches=2 if splits > 1 else 1)
+                   int(window or 0), int(keep_first), float(softcap or 0.0), _ptr(sinks), dtype_code(qkv.dtype), _stream(), launches=2 if splits > 1 else 1)
         return out
 
     # ------------------------------------------------------------------ a 32-bit stream with root-mean-square norms
@@ -1032,13 +1097,15 @@ class KernelLibrary:
                    _stream())
         return out
 
-    def sandwich_norm(self, stream: torch.Tensor, addend: torch.Tensor, post_w: torch.Tensor, post_eps: float, w: torch.Tensor, eps: float,
+    def sandwich_norm(self, stream: torch.Tensor, addend: torch.Tensor, post_w: torch.Tensor, post_eps: float, w: torch.Tensor | None, eps: float,
                       rows: torch.Tensor | None = None) -> torch.Tensor:
         """The float32 ``stream`` plus the root-mean-square norm of ``addend`` (activation dtype) under ``post_w``, written back unless
-        ``rows`` gathers; returns the norm of the sum under ``w`` in the addend's dtype."""
-        _need(stream, "stream", torch.float32); _need(addend, "addend"); _need(post_w, "post_w", torch.float32); _need(w, "w", torch.float32)
+        ``rows`` gathers; returns the norm of the sum under ``w`` in the addend's dtype (without ``w`` the sum itself, rounded)."""
+        _need(stream, "stream", torch.float32); _need(addend, "addend"); _need(post_w, "post_w", torch.float32)
+        if w is not None:
+            _need(w, "w", torch.float32)
         H = stream.shape[-1]
-        if addend.shape != stream.shape or post_w.numel() != H or w.numel() != H:
+        if addend.shape != stream.shape or post_w.numel() != H or (w is not None and w.numel() != H):
             raise KernelError("sandwich_norm: the stream, the addend and the weights differ in width")
         if rows is not None:
             _need(rows, "rows", torch.int32)
@@ -1222,6 +1289,33 @@ class KernelLibrary:
         self._call("roost_retention_scan_raw", _ptr(u), u.stride(0), 1 if activation == "silu" else 0, float(k_scale), _ptr(out), _ptr(state),
                    state.stride(0), _ptr(decay), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, _ptr(ws), dtype_code(u.dtype), _stream(),
                    launches=3 if ws is not None else 1)
+        return out
+
+    # ------------------------------------------------------------------ gated linear attention
+    def gla_scan(self, u, a_col: int, gate_w, gate_bias, tau: float, q_scale: float, state, q_indptr, slots, heads: int, dim: int, vdim: int,
+                 single: bool = False, chunked: bool | None = None) -> torch.Tensor:
+        """S <- diag(alpha) S + k v^T, o = S^T q a head over rows [q heads | k heads | v heads | ... a1 from ``a_col`` on] of ``u``, alpha =
+        sigmoid(a1 gate_w^T + gate_bias)^(1 / tau): float32 [T, heads * vdim]; see csrc/gated_linear_attention.cu. ``single``: every row brings
+        one token, the scan makes the decays itself. ``chunked`` None: steps of ``SCAN_CHUNKED_MIN_TOKENS`` tokens or more cut their rows into
+        chunks."""
+        _need_rows(u, "u"); _need(gate_w, "gate_w", u.dtype); _need(gate_bias, "gate_bias", torch.float32); _need(state, "state", torch.float32)
+        _need(q_indptr, "q_indptr", torch.int32); _need(slots, "slots", torch.int32)
+        T, (channels, rank) = u.shape[0], gate_w.shape
+        if channels != heads * dim or gate_bias.numel() != channels or u.shape[1] < max(heads * (2 * dim + vdim), a_col + rank):
+            raise KernelError("gla_scan: the rows or the decays' weights do not fit the sizes")
+        out = torch.empty((T, heads * vdim), dtype=torch.float32, device=u.device)
+        alpha = ws = ws_keep = None
+        if not single:
+            alpha = torch.empty((T, channels), dtype=torch.float32, device=u.device)
+            self._call("roost_gla_prepare", _ptr(u), u.stride(0), a_col, _ptr(gate_w), _ptr(gate_bias), _ptr(alpha), T, channels, rank, float(tau),
+                       dtype_code(u.dtype), _stream())
+            if (T >= self.SCAN_CHUNKED_MIN_TOKENS) if chunked is None else chunked:
+                chunks = self._lib.roost_gla_scan_chunks(T, slots.numel())
+                ws = torch.empty((chunks * heads * dim * vdim,), dtype=torch.float32, device=u.device)
+                ws_keep = torch.empty((chunks * channels,), dtype=torch.float32, device=u.device)
+        self._call("roost_gla_scan", _ptr(u), u.stride(0), float(q_scale), _ptr(alpha), a_col, _ptr(gate_w), _ptr(gate_bias), rank, float(tau), _ptr(out),
+                   _ptr(state), state.stride(0), _ptr(q_indptr), _ptr(slots), slots.numel(), T, heads, dim, vdim, _ptr(ws), _ptr(ws_keep),
+                   dtype_code(u.dtype), _stream(), launches=3 if ws is not None else 1)
         return out
 
     # ------------------------------------------------------------------ the recurrence whose gates read only the current token

@@ -29,11 +29,14 @@ class AttentionPlan:
     merge_work: torch.Tensor | None = None
 
 
-def attention_work(row_starts, row_counts, group: int, window: int | None, chunk: int, tile_rows: int = 64, cluster: int = 0):
+def attention_work(row_starts, row_counts, group: int, window: int | None, chunk: int, tile_rows: int = 64, cluster: int = 0,
+                   keep_first: int = 0):
     """(prefill pairs, decode quadruples, merge quadruples, slots) as flat int lists. ``chunk`` is a multiple of 64: a
     chunk starts on a boundary of the decode kernels' key tiles. With ``cluster`` = S > 0 a short row gets exactly S
     decode items (its chunks in key order, then empty ones) for a cluster of S CTAs that merges them itself: no merge
-    items and no slots."""
+    items and no slots. With ``keep_first`` (and a window) a row also has items for its request's first ``keep_first`` keys, whose first
+    key c is written as -1 - c (the kernels bound such an item by causality only); a row whose window still reaches them is listed like one
+    without a window, in items of that form."""
     if chunk <= 0 or chunk % 64:
         raise ValueError(f"decode chunk {chunk} is not a positive multiple of 64")
     prefill, decode, merge, tiles = [], [], [], []
@@ -46,20 +49,26 @@ def attention_work(row_starts, row_counts, group: int, window: int | None, chunk
             continue   # a padding row (see pad_row): no keys, no work
         if rows <= 16:
             lo = max(0, start - window + 1) if window else 0
-            first = (lo // chunk) * chunk
-            begins = range(first, kv_len, chunk)
-            if cluster:
-                if len(begins) > cluster:
-                    raise ValueError(f"a row of {kv_len} keys has {len(begins)} chunks of {chunk}: more than the cluster's {cluster}")
-                for r in range(cluster):
-                    c = first + r * chunk
-                    decode += [b, c, min(c + chunk, kv_len), r] if c < kv_len else [b, 0, 0, r]
-            elif len(begins) == 1:
-                decode += [b, first, min(first + chunk, kv_len), -1]
+            if keep_first and window:
+                if kv_len - window <= keep_first:       # the row's last token still sees every key
+                    ranges = [(-1 - c, min(c + chunk, kv_len)) for c in range(0, kv_len, chunk)]
+                else:
+                    ranges = [(-1 - c, min(c + chunk, keep_first)) for c in range(0, keep_first, chunk)]
+                    lo = max(lo, keep_first)
+                    ranges += [(c, min(c + chunk, kv_len)) for c in range(lo // chunk * chunk, kv_len, chunk)]
             else:
-                merge += [b, slots, len(begins) | (rows << 24), first_token]
-                for c in begins:
-                    decode += [b, c, min(c + chunk, kv_len), slots]
+                ranges = [(c, min(c + chunk, kv_len)) for c in range(lo // chunk * chunk, kv_len, chunk)]
+            if cluster:
+                if len(ranges) > cluster:
+                    raise ValueError(f"a row of {kv_len} keys has {len(ranges)} chunks of {chunk}: more than the cluster's {cluster}")
+                for r in range(cluster):
+                    decode += [b, *ranges[r], r] if r < len(ranges) else [b, 0, 0, r]
+            elif len(ranges) == 1:
+                decode += [b, *ranges[0], -1]
+            else:
+                merge += [b, slots, len(ranges) | (rows << 24), first_token]
+                for c, end in ranges:
+                    decode += [b, c, end, slots]
                     slots += 1
         else:
             for r0 in range(0, rows, tile_rows):
@@ -70,12 +79,22 @@ def attention_work(row_starts, row_counts, group: int, window: int | None, chunk
     return prefill, decode, merge, slots
 
 
+def kept_chunks(kv_cap: int, window: int, keep_first: int, chunk: int) -> int:
+    """The most decode items ``attention_work`` lists for a row of at most ``kv_cap`` keys and 16 tokens of a model that keeps its
+    first ``keep_first`` keys beside a window."""
+    kept = -(-keep_first // chunk)
+    return min(-(-max(kv_cap, 1) // chunk) + 1, -(-(window + 16) // chunk) + 1 + kept)
+
+
 def attention_caps(num_tokens: int, num_rows: int, kv_cap: int, group: int, chunk: int, tile_rows: int = 64,
-                   short_rows: bool = True, cluster: int = 0) -> tuple[int, int, int]:
+                   short_rows: bool = True, cluster: int = 0, window: int | None = None, keep_first: int = 0) -> tuple[int, int, int]:
     """Largest (prefill, decode, merge) item counts of a step of ``num_tokens`` tokens in ``num_rows`` rows whose
     requests hold at most ``kv_cap`` keys. A step of one token a row has work of one kind only; so has a step without
     ``short_rows`` (rows of at most 16 tokens, the only ones that can go to the decode kernel)."""
-    chunks = cluster if cluster else -(-kv_cap // chunk)
+    if cluster:
+        chunks = cluster
+    else:
+        chunks = kept_chunks(kv_cap, window, keep_first, chunk) if keep_first and window else -(-kv_cap // chunk)
     merges = 0 if cluster else num_rows
     if num_tokens == num_rows:
         if group > 16:
@@ -90,10 +109,10 @@ def _pad4(a: list) -> list:
 
 
 def plan_attention(row_starts, row_counts, group: int, window: int | None, chunk: int, device, tile_rows: int = 64,
-                   cluster: int = 0) -> AttentionPlan:
+                   cluster: int = 0, keep_first: int = 0) -> AttentionPlan:
     """The lists of one step on the device, for callers that run the attention kernels outside an engine (kernel tests,
     microbenchmarks)."""
-    prefill, decode, merge, slots = attention_work(row_starts, row_counts, group, window, chunk, tile_rows, cluster)
+    prefill, decode, merge, slots = attention_work(row_starts, row_counts, group, window, chunk, tile_rows, cluster, keep_first)
     plan = AttentionPlan(prefill_items=len(prefill) // 2, prefill_tile_rows=tile_rows, decode_items=len(decode) // 4, merge_items=len(merge) // 4, slots=slots,
                          merge_rows=max((z >> 24 for z in merge[2::4]), default=1), cluster_chunks=cluster)
     flat = _pad4(prefill) + _pad4(decode) + _pad4(merge)

@@ -41,7 +41,7 @@ class ParamDecl:
 class CacheNeed:
     """What one run of a mixer keeps between steps. ``paged``: ``planes`` tensors of ``kv_heads`` x ``head_dim`` per
     token (2: keys and values; 1: one vector a token, a latent from which a mixer makes both), every earlier token
-    (window None) or the last ``window`` tokens. ``state``: one tensor of ``state_shape`` per live request, zeroed when
+    (window None) or the last ``window`` tokens (and, with ``keep_first``, the request's first ``keep_first``). ``state``: one tensor of ``state_shape`` per live request, zeroed when
     the request's first token arrives."""
     kind: str                       # "paged" | "state"
     kv_heads: int = 0
@@ -50,6 +50,7 @@ class CacheNeed:
     planes: int = 2
     state_shape: tuple = ()
     state_dtype: torch.dtype = torch.float32
+    keep_first: int = 0
 
 
 class Runtime:

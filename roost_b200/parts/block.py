@@ -236,6 +236,59 @@ class SandwichWideBlock(Block):
         return norm.add_norm(h, residual.stream, rows=rows, post=residual.post)[0]
 
 
+class PostNormWideBlock(Block):
+    """x <- x + out_norm1(mixer(x)); x <- x + out_norm2(ff(x)) over a residual kept and summed in 32-bit: the only norms are those between a
+    sublayer's output and the sum. One kernel norms the output, adds it and hands the sum on, rounded to the activation dtype, to the
+    sublayer after it. The block hands on its last branch output and the residual with the norm still to be applied; ``close`` does the
+    last sum and the final norm of the wanted rows."""
+
+    def __init__(self, spec: BlockSpec, runtime: Runtime):
+        if spec.input_norm is not None or spec.post_mixer_norm is not None:
+            raise ValueError("post_norm_wide: sublayers read the stream as it is; the arrangement has no norm before them")
+        if spec.mixer_out_norm is None or (spec.feed_forward is not None and spec.feed_forward_out_norm is None):
+            raise ValueError("post_norm_wide: every sublayer needs the norm after it")
+        self.spec = spec
+        self.rt = runtime
+        self.mixer = MIXERS.build(spec.mixer, runtime)
+        self.mixer_out_norm = NORMS.build(spec.mixer_out_norm, runtime)
+        self.feed_forward = self.feed_forward_out_norm = None
+        if spec.feed_forward is not None:
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, runtime)
+            self.feed_forward_out_norm = NORMS.build(spec.feed_forward_out_norm, runtime)
+
+    def sub_parts(self):
+        parts = {"mixer": self.mixer, "mixer_out_norm": self.mixer_out_norm}
+        if self.feed_forward is not None:
+            parts.update({"feed_forward": self.feed_forward, "feed_forward_out_norm": self.feed_forward_out_norm})
+        return parts
+
+    @classmethod
+    def sub_specs(cls, spec: BlockSpec):
+        subs = {"mixer": (MIXERS, spec.mixer), "mixer_out_norm": (NORMS, spec.mixer_out_norm)}
+        if spec.feed_forward is not None:
+            subs.update({"feed_forward": (FEED_FORWARDS, spec.feed_forward), "feed_forward_out_norm": (NORMS, spec.feed_forward_out_norm)})
+        return subs
+
+    def __call__(self, h, residual, batch, cache, write_cache: bool = True):
+        if residual is None:
+            if h.dtype != torch.float32:
+                raise ValueError("post_norm_wide: the embedding must hand over a float32 stream")
+            stream = h
+            x = self.mixer_out_norm.round_stream(stream)
+        else:
+            stream = residual.stream
+            x = residual.post.join(h, stream)
+        a, post = self.mixer(x, batch, cache, write_cache), self.mixer_out_norm
+        if self.feed_forward is not None:
+            y = post.join(a, stream)
+            a, post = self.feed_forward(y, batch), self.feed_forward_out_norm
+        return a, NormedStream(stream, post)
+
+    def close(self, h, residual, norm, rows):
+        """The model's end: the last normed sum of the wanted rows and ``norm`` of it."""
+        return norm.add_norm(h, residual.stream, rows=rows, post=residual.post)[0]
+
+
 class StreamState:
     """The residual streams between two sublayers: the 32-bit tensor [tokens, streams, width] and the connection whose
     write-back of the branch output that travels beside it is still to be applied."""
@@ -308,6 +361,7 @@ class PreNormStreamsBlock(Block):
         return self._read(h, residual, None, norm, rows=rows)[0]
 
 
+register_block("post_norm_wide", PostNormWideBlock)
 register_block("sandwich_wide", SandwichWideBlock)
 register_block("pre_norm_streams", PreNormStreamsBlock)
 register_block("pre_norm_gated", PreNormGatedBlock)

@@ -109,6 +109,15 @@ class WideRmsNorm(Norm):
         return self.rt.kernels.wide_rms_norm(residual, None, self.spec.eps, self.rt.dtype, x, None, None), residual
 
 
+    def join(self, x: torch.Tensor, residual: torch.Tensor) -> torch.Tensor:
+        """residual + norm(x), which replaces ``residual`` in place; returns the sum in the activation dtype (one kernel)."""
+        return self.rt.kernels.sandwich_norm(residual, x, self.weight, self.spec.eps, None, self.spec.eps)
+
+    def round_stream(self, residual: torch.Tensor) -> torch.Tensor:
+        """The stream in the activation dtype, as a tensor of its own."""
+        return self.rt.kernels.wide_rms_norm(residual, None, self.spec.eps, self.rt.dtype)
+
+
 register_norm("rms_norm_wide", WideRmsNorm)
 register_norm("rms_norm", RmsNorm)
 register_norm("layer_norm", LayerNorm)

@@ -15,7 +15,7 @@ A second form of routing (``score`` "softmax", ``weight_on`` "output"): the scor
 the experts and the identity experts; a stored correction is added for the choice only; the weights are the chosen scores
 times a constant and multiply the experts' outputs; an identity expert has no weights and gives its input back; the shared
 expert's output is multiplied by the sigmoid of one more product a token, whose row rides along as the last row of the
-router's matrix. The experts' gate function and its limit are the spec's (``GatedMlpSpec``).
+router's matrix. With ``score`` "softmax_chosen" the weights are the softmax over the chosen logits alone. The experts' gate function and its limit are the spec's (``GatedMlpSpec``).
 """
 from __future__ import annotations
 
@@ -38,14 +38,16 @@ class RoutedMlp(FeedForward):
             raise ValueError("routed_mlp: more than 1024 experts or a top beyond 32 is more than the routing kernel serves")
         if s.activation not in GATE_FUNCTIONS:
             raise ValueError(f"routed_mlp: activation '{s.activation}' has no kernel (built: {', '.join(GATE_FUNCTIONS)})")
-        if (s.score, s.weight_on) not in (("sigmoid", "input"), ("softmax", "output")):
+        if (s.score, s.weight_on) not in (("sigmoid", "input"), ("softmax", "output"), ("softmax_chosen", "output")):
             raise ValueError(f"routed_mlp: score '{s.score}' with the weight on the {s.weight_on} has no kernel "
-                             "(built: sigmoid scores on the input, softmax scores on the output)")
+                             "(built: sigmoid scores on the input; softmax scores, over all or over the chosen, on the output)")
         if s.renormalize:
             raise ValueError("routed_mlp: renormalised weights have no kernel")
         self.legacy = s.score == "sigmoid"
         if self.legacy and (s.correction or s.identity_experts or s.shared_gate or s.route_scale != 1.0):
             raise ValueError("routed_mlp: a correction, identity experts, a scale or a gated shared expert need softmax scores on the output")
+        if s.correction and s.score != "softmax":
+            raise ValueError("routed_mlp: a correction belongs to softmax scores over all experts")
         if s.identity_experts < 0 or s.top > s.experts + s.identity_experts:
             raise ValueError("routed_mlp: top is more than the experts and identity experts together")
         if s.shared_gate and not s.shared_intermediate:
@@ -119,7 +121,7 @@ class RoutedMlp(FeedForward):
             ys = k.moe_expert_down(act, self.down, route)                       # [T * top, hidden]
             shared = self.shared(x, batch) if self.shared is not None else None
             return k.moe_combine(ys, route, shared)
-        route = k.moe_route(logits, s.top, score="softmax", correction=self.correction, scale=float(s.route_scale), routed=self.routed,
+        route = k.moe_route(logits, s.top, score=s.score, correction=self.correction, scale=float(s.route_scale), routed=self.routed,
                             real=s.experts)
         xs = k.moe_gather_scale(x, route, scale=False)                          # [T * top, hidden]: the rows, sorted by expert
         fn = dict(activation=s.activation, limit=float(s.limit))

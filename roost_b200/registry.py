@@ -57,7 +57,8 @@ def resolve(reader: ConfigReader) -> Architecture:
 
 
 def _register_builtin() -> None:
-    from .config import lafanex, lovurax, nomivik, qwen3, revirax, vamatar
+    from .config import lafanex, lovurax, nomivik, qwen3, revirax, vamatar, zufusun
+    register_architecture(zufusun.ARCHITECTURE, read_config=zufusun.ZufusunConfig.from_reader, to_spec=lambda cfg, tied=None: cfg.to_spec(tied))
     register_architecture(revirax.ARCHITECTURE, read_config=revirax.ReviraxConfig.from_reader, to_spec=lambda cfg, tied=None: cfg.to_spec(tied))
     register_architecture(lovurax.ARCHITECTURE, read_config=lovurax.LovuraxConfig.from_reader, to_spec=lambda cfg, tied=None: cfg.to_spec(tied))
     register_architecture(nomivik.ARCHITECTURE, read_config=nomivik.NomivikConfig.from_reader, to_spec=lambda cfg, tied=None: cfg.to_spec(tied))

@@ -66,6 +66,21 @@ def checkpoint_has(model_dir, name: str) -> bool:
         return name in st.entries
 
 
+def checkpoint_shapes(model_dir) -> dict[str, tuple]:
+    """Tensor name -> shape of what the checkpoint holds ({} for a folder without one), for sizes that no configuration key gives."""
+    model_dir = Path(model_dir)
+    if not (model_dir / "model.safetensors").exists() and not (model_dir / "model.safetensors.index.json").exists():
+        return {}
+    shapes = {}
+    for f in checkpoint_files(model_dir):
+        try:
+            with SafetensorsFile(f) as st:
+                shapes.update({n: tuple(e.shape) for n, e in st.entries.items()})
+        except SafetensorsError as e:
+            raise WeightError(str(e)) from None
+    return shapes
+
+
 def expected_tensors(decls: dict, names: dict) -> dict[str, tuple]:
     """Checkpoint tensor name -> shape, from the parts' declarations and the architecture's name map."""
     out = {}

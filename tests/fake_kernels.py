@@ -118,33 +118,42 @@ class FakeKernels:
         return out
 
     # ---- latent attention
-    def latent_prepare(self, q, down, pool, latent_w, inv_freq, rotary_dim, positions, slot_mapping, heads, nope, rope, rank, eps, page_size):
-        T = q.shape[0]
+    def latent_prepare(self, q, down, pool, latent_w, inv_freq, rotary_dim, positions, slot_mapping, heads, nope, rope, rank, eps, page_size,
+                       interleaved=False, cq=None, cq_w=None):
+        T = positions.numel()
         half = rotary_dim // 2
+        first, second = (slice(0, rotary_dim, 2), slice(1, rotary_dim, 2)) if interleaved else (slice(0, half), slice(half, rotary_dim))
         if inv_freq is None:      # no rotated part
             inv_freq = torch.zeros(0, dtype=torch.float64)
         ang = positions.double()[:, None] * inv_freq[None, :]
         c, s = torch.cos(ang).float(), torch.sin(ang).float()
 
         def turn(v):        # [..., rope] float32, rotated in its first rotary_dim elements
-            u, w2 = v[..., :half].clone(), v[..., half:rotary_dim].clone()
+            u, w2 = v[..., first].clone(), v[..., second].clone()
             shape = [T] + [1] * (v.dim() - 2) + [half]
-            v[..., :half] = u * c.reshape(shape) - w2 * s.reshape(shape)
-            v[..., half:rotary_dim] = w2 * c.reshape(shape) + u * s.reshape(shape)
+            v[..., first] = u * c.reshape(shape) - w2 * s.reshape(shape)
+            v[..., second] = w2 * c.reshape(shape) + u * s.reshape(shape)
             return v
 
-        qv = q.view(T, heads, nope + rope)
-        qv[:, :, nope:] = turn(qv[:, :, nope:].float()).to(q.dtype)
+        cq_out = None
+        if cq is not None:
+            f = cq.float()
+            cq_out = (f * torch.rsqrt((f * f).mean(-1, keepdim=True) + eps) * cq_w).to(cq.dtype)
+        if q is not None:
+            qv = q.view(T, heads, nope + rope)
+            qv[:, :, nope:] = turn(qv[:, :, nope:].float()).to(q.dtype)
         if down is not None:
             lat = down[:, :rank].float()
             lat = lat * torch.rsqrt((lat * lat).mean(-1, keepdim=True) + eps) * latent_w
-            entry = torch.cat([lat, turn(down[:, rank:].float())], -1).to(pool.dtype)
+            entry = torch.cat([lat, turn(down[:, rank:].float().clone())], -1).to(pool.dtype)
             for t in range(T):
                 slot = int(slot_mapping[t])
                 if slot >= 0:
                     pool[slot // page_size, 0, slot % page_size] = entry[t]
+        return cq_out
 
-    def latent_attention(self, q_latent, q, pool, positions, token_row, kv_indptr, kv_indices, heads, nope, rope, rank, scale, window, kv_cap=0, few_rows=False, q_indptr=None):
+    def latent_attention(self, q_latent, q, pool, positions, token_row, kv_indptr, kv_indices, heads, nope, rope, rank, scale, window, kv_cap=0, few_rows=False, q_indptr=None,
+                         sinks=None):
         T = q.shape[0]
         page = pool.shape[2]
         out = torch.zeros(heads, T, rank, dtype=q.dtype)
@@ -157,7 +166,9 @@ class FakeKernels:
             lo = max(0, pos - window + 1) if window else 0
             e = torch.stack([pool[int(pages[j // page]), 0, j % page] for j in range(lo, pos + 1)]).float()    # [n, rank + rope]
             sc = (q_latent[:, t].float() @ e[:, :rank].T + qr[t] @ e[:, rank:].T) * scale                    # [heads, n]
-            out[:, t] = (torch.softmax(sc, -1) @ e[:, :rank]).to(q.dtype)
+            if sinks is not None:       # one more key, of the stored score, whose weight nobody takes
+                sc = torch.cat([sc, sinks[:, None]], -1)
+            out[:, t] = (torch.softmax(sc, -1)[:, : e.shape[0]] @ e[:, :rank]).to(q.dtype)
         return out
 
     # ---- mamba-2
@@ -225,6 +236,10 @@ class FakeKernels:
         if score == "sigmoid":
             s = torch.sigmoid(logits)
             choice = logits                          # by logit: the sigmoid saturates in 32-bit
+        elif score == "softmax_chosen":
+            choice = logits[:, :E].float()
+            s = torch.exp(choice - choice.max(-1, keepdim=True).values)
+            s = s / torch.topk(s, top, dim=-1).values.sum(-1, keepdim=True) * scale
         else:
             s = torch.softmax(logits[:, :E].float(), dim=-1)
             choice = s + (correction.float() if correction is not None else 0.0)
@@ -390,7 +405,48 @@ class FakeKernels:
             stream.copy_(s)
         else:
             s = s[rows.long()]
-        return (s * torch.rsqrt((s * s).mean(-1, keepdim=True) + eps) * w).to(addend.dtype)
+        return (s * torch.rsqrt((s * s).mean(-1, keepdim=True) + eps) * w if w is not None else s).to(addend.dtype)
+
+    def gla_scan(self, u, a_col, gate_w, gate_bias, tau, q_scale, state, q_indptr, slots, heads, dim, vdim, single=False, chunked=None):
+        T, QK, R = u.shape[0], heads * dim, gate_w.shape[1]
+        f = u.float()
+        alpha = torch.exp(torch.nn.functional.logsigmoid(f[:, a_col : a_col + R] @ gate_w.float().T + gate_bias) / tau).reshape(T, heads, dim)
+        q, k = f[:, :QK].reshape(T, heads, dim) * q_scale, f[:, QK : 2 * QK].reshape(T, heads, dim)
+        v = f[:, 2 * QK : 2 * QK + heads * vdim].reshape(T, heads, vdim)
+        out = torch.zeros(T, heads, vdim)
+        for r in range(slots.numel()):
+            slot = int(slots[r])
+            S = state[slot, : QK * vdim].reshape(heads, dim, vdim).clone()
+            for t in range(int(q_indptr[r]), int(q_indptr[r + 1])):
+                S = alpha[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+                out[t] = (q[t][:, :, None] * S).sum(1)
+            if int(q_indptr[r + 1]) > int(q_indptr[r]):
+                state[slot, : QK * vdim] = S.reshape(-1)
+        return out.reshape(T, heads * vdim)
+
+    def sink_attention_prepare_normed(self, qkv, k_pool, v_pool, slot_mapping, heads, kv_heads, dim, vdim, q_w, k_w, eps, page_size, q_out=None):
+        T, Q, K = qkv.shape[0], heads * dim, kv_heads * dim
+
+        def norm(x, w):
+            x = x.float()
+            return (x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * w).to(qkv.dtype)
+
+        k = norm(qkv[:, Q : Q + K], k_w).reshape(T, kv_heads, dim)
+        v = qkv[:, Q + K : Q + K + kv_heads * vdim].reshape(T, kv_heads, vdim)
+        q = norm(qkv[:, :Q], q_w)
+        if q_out is not None:
+            q_out.copy_(q.reshape(T, heads, dim))
+        else:
+            qkv[:, :Q] = q
+        for t in range(T):
+            slot = int(slot_mapping[t])
+            if slot < 0:
+                continue
+            page, off = divmod(slot, page_size)
+            if v_pool is None:
+                k_pool[page, :, off] = torch.cat([k[t], v[t]], -1)
+            else:
+                k_pool[page, :, off], v_pool[page, :, off] = k[t], v[t]
 
     def weighted_sum(self, xs, ws):
         return sum(float(w) * x.float() for w, x in zip(ws, xs)).to(xs[0].dtype)
@@ -399,7 +455,7 @@ class FakeKernels:
         return (torch.clamp(x.float(), min=0.0) ** 2).to(x.dtype)
 
     def sink_attention(self, qkv, k_pool, v_pool, positions, token_row, kv_indptr, kv_indices, heads, kv_heads, dim, vdim, scale, sink, kv_cap=0,
-                       window=None, softcap=0.0, sinks=None):
+                       window=None, softcap=0.0, sinks=None, keep_first=0):
         T = qkv.shape[0]
         page_size = k_pool.shape[2]
         out = torch.zeros(T, heads * vdim, dtype=qkv.dtype)
@@ -411,14 +467,12 @@ class FakeKernels:
             r = int(token_row[t])
             pages = kv_indices[int(kv_indptr[r]) : int(kv_indptr[r + 1])].long()
             lo = max(0, pos - window + 1) if window else 0
-            first_page = lo // page_size            # pages before it may have been given back (entry -1): never touched
-            pages, lo = pages[first_page:], lo - first_page * page_size
-            hi = pos + 1 - first_page * page_size
-            entries = k_pool[pages].permute(1, 0, 2, 3).reshape(kv_heads, -1, k_pool.shape[3])[:, lo:hi].float()
+            seen = torch.tensor(list(range(min(keep_first, lo))) + list(range(lo, pos + 1)))
+            at_page, at_off = pages[seen // page_size], seen % page_size        # pages nobody sees may have been given back (entry -1)
+            assert (at_page >= 0).all(), "a page that a query sees was given back"
+            entries = k_pool[at_page, :, at_off].permute(1, 0, 2).float()
             keys = entries[..., :dim]
-            vals = (entries[..., dim:] if v_pool is None
-                    else v_pool[pages].permute(1, 0, 2, 3).reshape(kv_heads, -1, vdim)[:, lo:hi].float())
-            assert (pages[lo // page_size :] >= 0).all(), "a page inside the window was given back"
+            vals = entries[..., dim:] if v_pool is None else v_pool[at_page, :, at_off].permute(1, 0, 2).float()
             q = qkv[t, : heads * dim].float().reshape(heads, dim)
             for h in range(heads):
                 s = (keys[h // group] @ q[h]) * scale
