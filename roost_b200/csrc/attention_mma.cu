@@ -577,6 +577,7 @@ __global__ void __launch_bounds__(NWARPS * 32)
     if (pr < rows_total) {
       qpos[r] = pos0 + pr / group;
       qlo[r] = window > 0 && windowed ? max(keep_first, qpos[r] - window + 1) : 0;
+      if (!windowed) qpos[r] = min(qpos[r], kv_end - 1);       // such a range may end in the middle of a tile
     } else {
       qpos[r] = -1;
       qlo[r] = 0;
@@ -999,6 +1000,7 @@ __global__ void __launch_bounds__((kTmaConsumers + 1) * 32, 2)
       if (pr < rows_total) {
         qpos[r] = pos0 + pr / group;
         qlo[r] = window > 0 && c.windowed ? max(keep_first, qpos[r] - window + 1) : 0;
+        if (!c.windowed) qpos[r] = min(qpos[r], c.hi);         // such a range may end in the middle of a tile
       } else {
         qpos[r] = -1;
         qlo[r] = 0;

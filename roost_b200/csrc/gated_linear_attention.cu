@@ -16,6 +16,8 @@
 // with S'; a state S before the chunk is P S + S' after it, P the products of the chunk's decays a channel. The first walk leaves every
 // chunk's own S' and P, one thread an entry then carries the row's state from chunk to chunk leaving every chunk's true starting state
 // in the place of S', and a second walk of every chunk from there writes the outputs and, from a row's last chunk, the slot.
+//
+// What an earlier kernel of the step writes comes through pointers without __restrict__: with it the compiler may load before pdl_wait().
 #include "common.cuh"
 
 namespace roost {
@@ -29,7 +31,7 @@ __device__ __forceinline__ float gla_decay(float z, float inv_tau) {
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) gla_prepare_kernel(const T* __restrict__ u, int64_t ld, int a_col, const T* __restrict__ w,
+__global__ void __launch_bounds__(256) gla_prepare_kernel(const T* u, int64_t ld, int a_col, const T* __restrict__ w,
                                                          const float* __restrict__ bias, float* __restrict__ alpha, int tokens, int channels, int rank,
                                                          float inv_tau) {
   extern __shared__ float rows[];      // [kGlaPrepareTokens][rank]
@@ -86,8 +88,8 @@ struct GlaGate {
 // in ws[chunk] and, from the first slice of columns, P in ws_keep[chunk]; a row's last chunk is skipped. MODE 2: a warp walks one chunk
 // from ws[chunk] (the carry kernel put the chunk's true starting state there) and writes the outputs; a row's last chunk writes the slot.
 template <typename T, int DREG, int MODE>
-__global__ void __launch_bounds__(32) gla_scan_kernel(const T* __restrict__ u, int64_t ld, float q_scale, const float* __restrict__ alpha, GlaGate<T> gate,
-                                                     float* __restrict__ out, float* state, int64_t state_stride, const int32_t* __restrict__ q_indptr,
+__global__ void __launch_bounds__(32) gla_scan_kernel(const T* u, int64_t ld, float q_scale, const float* alpha, GlaGate<T> gate,
+                                                     float* out, float* state, int64_t state_stride, const int32_t* __restrict__ q_indptr,
                                                      const int32_t* __restrict__ slots, int rows, int heads, int dim, int vdim, float* ws, float* ws_keep) {
   extern __shared__ float4 sm4[];    // two staging slots of dim (k, q, alpha, -); then S when it does not live in registers
   constexpr int NREG = DREG > 0 ? DREG : 1;
@@ -201,7 +203,7 @@ __global__ void __launch_bounds__(32) gla_scan_kernel(const T* __restrict__ u, i
 // One thread an entry of S of a (row, head): the row's state through its chunks in order. ws[chunk] holds the chunk's own S' on entry
 // (all but a row's last chunk) and the state the chunk starts from on exit; ws_keep[chunk] the decays' products a channel. The slot is
 // read, not written.
-__global__ void gla_carry_kernel(const float* state, int64_t state_stride, float* ws, const float* __restrict__ ws_keep,
+__global__ void gla_carry_kernel(const float* state, int64_t state_stride, float* ws, const float* ws_keep,
                                  const int32_t* __restrict__ q_indptr, const int32_t* __restrict__ slots, int heads, int dim, int vdim) {
   pdl_launch_dependents();
   pdl_wait();

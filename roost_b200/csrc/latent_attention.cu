@@ -26,10 +26,10 @@ constexpr int kLaWarps = 8;
 constexpr int kLaMaxRank = 1024;
 
 template <typename T>
-__global__ void latent_prepare_kernel(T* q, const T* __restrict__ down, T* pool, const float* __restrict__ latent_w,
+__global__ void latent_prepare_kernel(T* q, const T* down, T* pool, const float* __restrict__ latent_w,
                                       const double* __restrict__ inv_freq, const int32_t* __restrict__ positions,
                                       const int32_t* __restrict__ slot_mapping, int heads, int nope, int rope, int rot_dims, int rank, float eps,
-                                      int interleaved, int64_t ld_down, const T* __restrict__ cq, T* __restrict__ cq_out, const float* __restrict__ cq_w,
+                                      int interleaved, int64_t ld_down, const T* cq, T* cq_out, const float* __restrict__ cq_w,
                                       int q_rank) {
   extern __shared__ float sm[];      // rot_dims/2 cosines, rot_dims/2 sines, 32 floats of scratch
   const int half = rot_dims / 2;

@@ -128,7 +128,8 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
     __syncwarp();
   }
   if (mode == 2) {
-    const float e = lane < top ? expf(chosen - __shfl_sync(0xffffffffu, chosen, 0)) : 0.f;     // the first choice is the largest
+    const float largest = __shfl_sync(0xffffffffu, chosen, 0);       // the first choice's logit; every lane takes part in the shuffle
+    const float e = lane < top ? expf(chosen - largest) : 0.f;
     const float sum = warp_sum(e);
     if (lane < top) pair_weight[(size_t)t * top + lane] = e / sum * scale;
   }

@@ -94,9 +94,10 @@ __global__ void wide_rms_norm_kernel(float* stream, const T* __restrict__ addend
 
 // The norm after a sublayer and the norm before the next one in one pass over a 32-bit stream. One block per output row: the addend's
 // root mean square, s = stream + addend * inv * post_w (written back unless the rows are gathered), then s's root mean square and the
-// output, rounded once. Without w the output is s itself, rounded once (a next sublayer that reads the stream as it is). Rows a block covers with eight numbers a thread stay in registers (VEC); others go through shared memory.
+// output, rounded once. Without w the output is s itself, rounded once (a next sublayer that reads the stream as it is). `addend` carries
+// no __restrict__: with it the compiler may load the row before pdl_wait(), while the kernel that writes it is still running. Rows a block covers with eight numbers a thread stay in registers (VEC); others go through shared memory.
 template <typename T, bool VEC>
-__global__ void sandwich_norm_kernel(float* stream, const T* __restrict__ addend, const float* __restrict__ post_w, float post_eps,
+__global__ void sandwich_norm_kernel(float* stream, const T* addend, const float* __restrict__ post_w, float post_eps,
                                      const float* __restrict__ w, T* __restrict__ out, const int32_t* __restrict__ rows, int hidden, float eps) {
   extern __shared__ float row[];  // 32 floats of reduction scratch; without VEC `hidden` floats after them
   float* scratch = row;
