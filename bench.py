@@ -633,6 +633,61 @@ def revirax_main(args) -> int:
     return 0
 
 
+# Zufusun models at the same widths, depths, vocabularies and expert sizes (no shared expert), every layer with routed experts: of every four
+# layers one latent attention (a query latent, its own key/value latent or, every other time, the last one's), one grouped attention with
+# joined query and key norms under a window beside 64 first tokens, two gated linear attentions (heads of 64 keys and 128 values, as wide in
+# values as the model). The Vamatar model beside each is the closest design the engine has: latent attention, recurrences with a matrix
+# state a head, routed experts, a 32-bit stream.
+def _zufusun_config(width, heads, dim, rot, vdim, rank, window, experts, top, ff, layers, vocab, **_):
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": 3 * rank // 2, "kv_rank": rank, "rot": {"base": 1000000.0, "dims": rot},
+              "scale": (dim + rot) ** -0.5}
+    attention = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                "mask": {"size": window // 2, "keep_first": 64}}}
+    gla = {"type": "gla", "mixer": {"heads": width // 128, "dim": 64, "vdim": 128, "tau": 16.0}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": 7.0}}
+    out, owner = [], None
+    for i in range(layers):
+        if i % 4 == 0:
+            mixer = dict(latent) if (i // 4) % 2 == 0 else dict(latent, kv_from=owner)
+            owner = i if (i // 4) % 2 == 0 else owner
+            out.append({"type": "latent_attention", "mixer": mixer, "mlp": moe})
+        else:
+            out.append(dict(attention if i % 4 == 2 else gla, mlp=moe))
+    return {"architecture": "Zufusun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": out}
+
+
+def zufusun_main(args) -> int:
+    """Prefill and decode throughput of Zufusun models beside Vamatar models (the closest design the engine has) of equal width, depth,
+    vocabulary and expert sizes, one JSON line."""
+    import torch
+
+    from roost_b200.config.zufusun import ZufusunConfig
+    pk, pk_src = peaks()
+    out = {}
+    for name in args.design_sizes.split(","):
+        s = DESIGN_SIZES[name]
+        rec = {}
+        for which in ("zufusun", "vamatar"):
+            model, _ = build_from_config(ZufusunConfig, _zufusun_config(**s), torch.bfloat16) if which == "zufusun" else build_vamatar(s, torch.bfloat16)
+            r = {"weight_gb": round(model.weight_bytes() / 1e9, 3)}
+            ms = timed_prefill(model, args.prefill_tokens)
+            r["prefill"] = {"tokens": args.prefill_tokens, "ms": round(ms, 3), "tokens_per_s": round(args.prefill_tokens / ms * 1e3)}
+            for batch in _ints(args.design_batches):
+                tps, ms, launches, _ = timed_decode(model, batch, args.design_context, args.steps, max(args.warmup, 3))
+                r[f"decode_b{batch}"] = {"context": args.design_context, "ms": round(ms, 4), "tokens_per_s": round(tps), "launches": launches[0] // args.steps,
+                                         "library_launches": launches[1] // args.steps}
+            rec[which] = r
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+        rec["config"] = s
+        out[name] = rec
+    print(json.dumps({"metric": "prefill and decode tokens/s of Zufusun models beside Vamatar models of equal width, depth, vocabulary and expert sizes",
+                      "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "impl": "ours", "peaks": pk_src,
+                      "data": "synthetic: seeded random weights, seeded random tokens; device-timed with CUDA events", "sizes": out}))
+    return 0
+
+
 def designs_main(args) -> int:
     """Prefill and decode throughput of Vamatar models beside Qwen3-shaped models of equal size, one JSON line."""
     import torch
@@ -644,6 +699,8 @@ def designs_main(args) -> int:
         return lovurax_main(args)
     if args.design == "revirax":
         return revirax_main(args)
+    if args.design == "zufusun":
+        return zufusun_main(args)
     pk, pk_src = peaks()
     out = {}
     for name in args.design_sizes.split(","):
@@ -692,8 +749,8 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=0, help="layers built (default: all the layers of --sizes)")
     ap.add_argument("--sizes", default="8b", choices=sorted(SIZES), help="whose layer sizes: Qwen3-0.6B, -8B (the headline) or -32B")
     ap.add_argument("--design-sizes", default="w1024,w2048", help="--workload designs: which of the Vamatar layer sizes to measure")
-    ap.add_argument("--design", default="vamatar", choices=["vamatar", "lafanex", "nomivik", "lovurax", "revirax"],
-                    help="--workload designs: vamatar (beside Qwen3-shaped models), lafanex (beside Vamatar models of equal size) or "
+    ap.add_argument("--design", default="vamatar", choices=["vamatar", "lafanex", "nomivik", "lovurax", "revirax", "zufusun"],
+                    help="--workload designs: vamatar (beside Qwen3-shaped models), lafanex or zufusun (beside Vamatar models of equal size) or "
                          "nomivik (beside Lafanex models with dense feed-forwards of equal size) or lovurax or revirax (beside Nomivik models of "
                          "equal size)")
     ap.add_argument("--design-batches", default="1,8", help="--workload designs: decode batch sizes")

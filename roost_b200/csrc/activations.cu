@@ -71,6 +71,24 @@ __global__ void head_gate_mul_kernel(T* __restrict__ x, const T* __restrict__ g,
   }
 }
 
+// The same with a gate a number (heads of one value), 16 bytes a thread; a block a token. x and g come from earlier kernels: no __restrict__,
+// with which the compiler may load them before pdl_wait().
+template <typename T>
+__global__ void element_gate_mul_kernel(T* x, const T* g, int64_t ld_g, int col, int n) {
+  constexpr int V = Vec<T>::N;
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+    float a[V], b[V];
+    Vec<T>::load(x + t * n + i, a);
+    Vec<T>::load(g + t * ld_g + col + i, b);
+#pragma unroll
+    for (int j = 0; j < V; ++j) a[j] *= sigmoid_f(b[j]);
+    Vec<T>::store(x + t * n + i, a);
+  }
+}
+
 }  // namespace roost
 
 using namespace roost;
@@ -109,6 +127,13 @@ extern "C" int roost_head_gate_mul(void* x, const void* g, int64_t ld_g, int col
   ROOST_REQUIRE(tokens >= 0 && heads > 0 && vdim > 0 && col >= 0 && ld_g >= col + heads, "head_gate_mul: sizes do not fit");
   ROOST_REQUIRE(x && g, "head_gate_mul: a pointer is null");
   if (tokens == 0) return ROOST_OK;
+  const int vec = dtype == ROOST_F32 ? 4 : 8;
+  if (vdim == 1 && heads % vec == 0 && col % vec == 0 && ld_g % vec == 0 && ((uintptr_t)x | (uintptr_t)g) % 16 == 0) {
+    const int wide = heads / vec >= 256 ? 256 : (heads / vec >= 128 ? 128 : 64);
+    ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(element_gate_mul_kernel<T>, dim3(tokens), dim3(wide), 0, (cudaStream_t)stream, (T*)x, (const T*)g, ld_g, col,
+                                                 heads));
+    return check_launch("head_gate_mul");
+  }
   const int threads = heads * vdim >= 1024 ? 256 : 128;
   ROOST_DISPATCH_DTYPE(dtype, T, launch_kernel(head_gate_mul_kernel<T>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, (T*)x, (const T*)g, ld_g, col,
                                                heads, vdim));

@@ -8,9 +8,12 @@
 //
 // prepare: alpha of every token as float32 [tokens, heads * dim]; a thread a channel, whose row of W it reads once for 8 tokens.
 //
-// scan: one warp (a block) per (row, head, 32 columns of S). A lane keeps its column of S in registers (dim up to 128) or in shared
-// memory (beyond); a token's (k, q, alpha) are staged in shared memory once and read by all lanes; the next token's inputs are loaded
-// while the current one is multiplied. A step of one token a row forms its decays in the scan itself (alpha null): no prepare kernel.
+// scan, heads of up to 128 keys: a block of W warps per (row, head, 32 W columns of S), a warp 32 columns. Lane (cg, dg) of a warp keeps the
+// entries of four columns 4 cg .. 4 cg + 3 and of the keys d = 4 i + dg in registers, so that a staged (k, q, alpha), read by all lanes of its
+// dg at once, serves four columns; S^T q is the sum over a quad's four lanes. The next 2 W tokens' inputs travel from memory to registers
+// while the current ones are multiplied, and are widened to 32-bit on their way into the other half of the stage. Wider heads: one warp
+// (a block) per (row, head, 32 columns), S in shared memory, inputs one token ahead. A step of one token a row forms its decays in the scan
+// itself (alpha null): no prepare kernel.
 //
 // Steps of many tokens cut every row into chunks of 64 tokens that run side by side (three launches): a chunk walked from S = 0 ends
 // with S'; a state S before the chunk is P S + S' after it, P the products of the chunk's decays a channel. The first walk leaves every
@@ -19,6 +22,8 @@
 //
 // What an earlier kernel of the step writes comes through pointers without __restrict__: with it the compiler may load before pdl_wait().
 #include "common.cuh"
+
+#include <type_traits>
 
 namespace roost {
 
@@ -83,17 +88,175 @@ struct GlaGate {
   float inv_tau;
 };
 
-// DREG > 0: S in registers, dim <= DREG. DREG == 0: S in shared memory after the staging area, [dim][32].
-// MODE 0: a warp walks its row's tokens from the slot and writes the slot back. MODE 1: a warp walks one chunk from S = 0 and leaves S'
-// in ws[chunk] and, from the first slice of columns, P in ws_keep[chunk]; a row's last chunk is skipped. MODE 2: a warp walks one chunk
-// from ws[chunk] (the carry kernel put the chunk's true starting state there) and writes the outputs; a row's last chunk writes the slot.
-template <typename T, int DREG, int MODE>
+// MODE 0: a row's tokens from the slot, which is written back. MODE 1: one chunk from S = 0, leaving S' in ws[chunk] and, from the first
+// columns' block, P in ws_keep[chunk]; a row's last chunk is skipped. MODE 2: one chunk from ws[chunk] (the carry kernel put the chunk's true
+// starting state there), writing the outputs; a row's last chunk writes the slot.
+template <typename T, int DREG, int W, int MODE>
+__global__ void __launch_bounds__(32 * W) gla_tile_kernel(const T* u, int64_t ld, float q_scale, const float* alpha, GlaGate<T> gate, float* out, float* state,
+                                                         int64_t state_stride, const int32_t* __restrict__ q_indptr, const int32_t* __restrict__ slots,
+                                                         int rows, int heads, int dim, int vdim, float* ws, float* ws_keep) {
+  constexpr int NT = 32 * W, TT = 2 * W, DG = DREG / 4, NE = TT * DREG / NT;
+  __shared__ float4 kqa[2][TT][DREG];
+  __shared__ __align__(16) float vs[2][TT][NT];
+  __shared__ float products[NT > DREG ? NT : DREG];
+  pdl_launch_dependents();
+  int r = blockIdx.x, k = 0, chunks_of_row = 1;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dg = lane & 3, cg = lane >> 2;
+  if (MODE != 0 && !gla_chunk_of_block(q_indptr, rows, blockIdx.x, r, k, chunks_of_row)) return;
+  if (MODE == 1 && k == chunks_of_row - 1) return;       // nobody starts from the state a row's last chunk ends with
+  int start = q_indptr[r], end = q_indptr[r + 1];
+  if (MODE != 0) {
+    start += k * kGlaChunkTokens;
+    end = min(end, start + kGlaChunkTokens);
+  }
+  const size_t head_state = (size_t)dim * vdim;
+  float* slot = state + (size_t)slots[r] * state_stride + (size_t)h * head_state;
+  float* wsh = MODE != 0 ? ws + ((size_t)blockIdx.x * heads + h) * head_state : nullptr;
+  const float* hs = MODE == 0 ? slot : wsh;
+  const int QK = heads * dim;
+  const int col_block = blockIdx.z * NT, col0 = col_block + warp * 32 + cg * 4;
+  const bool wide = (vdim & 3) == 0 && ((uintptr_t)slot & 15) == 0 && (MODE == 0 || ((uintptr_t)wsh & 15) == 0);      // four columns at a time
+  pdl_wait();
+  if (end <= start) return;
+  float S[DG][4];
+#pragma unroll
+  for (int i = 0; i < DG; ++i) {
+    const int d = 4 * i + dg;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) S[i][c] = 0.f;
+    if (MODE != 1 && d < dim) {
+      const float* src = hs + (size_t)d * vdim + col0;
+      if (wide && col0 < vdim) {
+        const float4 v = *reinterpret_cast<const float4*>(src);
+        S[i][0] = v.x; S[i][1] = v.y; S[i][2] = v.z; S[i][3] = v.w;
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (col0 + c < vdim) S[i][c] = src[c];
+      }
+    }
+  }
+  // the next stage's inputs on their way: entries e = tid + j NT of [TT tokens][DREG keys], and column tid of every token's values
+  float nk[NE], nq[NE], na[NE], nv[TT], prod = 1.0f;
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int j = 0; j < NE; ++j) {
+      const int e = tid + j * NT, t = t0 + e / DREG, d = e % DREG;
+      nk[j] = nq[j] = na[j] = 0.f;
+      if (t < end && d < dim) {
+        const T* row = u + (size_t)t * ld;
+        const int c = h * dim + d;
+        nq[j] = to_float(row[c]);
+        nk[j] = to_float(row[QK + c]);
+        if (MODE != 0 || alpha != nullptr) {
+          na[j] = alpha[(size_t)t * QK + c];
+        } else {
+          float z = 0.f;
+          for (int i = 0; i < gate.rank; ++i) z = fmaf(to_float(row[gate.a_col + i]), to_float(gate.w[(size_t)c * gate.rank + i]), z);
+          na[j] = gla_decay(z + gate.bias[c], gate.inv_tau);
+        }
+        if (MODE == 1) prod *= na[j];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < TT; ++j) {
+      const int t = t0 + j;
+      nv[j] = t < end && col_block + tid < vdim ? to_float(u[(size_t)t * ld + 2 * QK + (size_t)h * vdim + col_block + tid]) : 0.f;
+    }
+  };
+  auto store = [&](int buf) {
+#pragma unroll
+    for (int j = 0; j < NE; ++j) {
+      const int e = tid + j * NT;
+      kqa[buf][e / DREG][e % DREG] = make_float4(nk[j], nq[j] * q_scale, na[j], 0.f);
+    }
+#pragma unroll
+    for (int j = 0; j < TT; ++j) vs[buf][j][tid] = nv[j];
+  };
+  fetch(start);
+  store(0);
+  __syncthreads();
+  const bool live = col_block + warp * 32 < vdim;        // the warp has columns
+  int buf = 0;
+  for (int t0 = start; t0 < end; t0 += TT, buf ^= 1) {
+    const bool more = t0 + TT < end;
+    if (more) fetch(t0 + TT);
+    if (live) {
+      const int n = min(TT, end - t0);
+      for (int tt = 0; tt < n; ++tt) {
+        const float4 v = *reinterpret_cast<const float4*>(&vs[buf][tt][warp * 32 + cg * 4]);
+        float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
+#pragma unroll
+        for (int i = 0; i < DG; ++i) {
+          const float4 f = kqa[buf][tt][4 * i + dg];
+          S[i][0] = fmaf(f.z, S[i][0], f.x * v.x);
+          S[i][1] = fmaf(f.z, S[i][1], f.x * v.y);
+          S[i][2] = fmaf(f.z, S[i][2], f.x * v.z);
+          S[i][3] = fmaf(f.z, S[i][3], f.x * v.w);
+          if (MODE != 1) {
+            o0 = fmaf(S[i][0], f.y, o0);
+            o1 = fmaf(S[i][1], f.y, o1);
+            o2 = fmaf(S[i][2], f.y, o2);
+            o3 = fmaf(S[i][3], f.y, o3);
+          }
+        }
+        if (MODE != 1) {
+          // the quad's sums of four columns, one column left in each lane: lane dg ends with column dg
+          const bool b0 = dg & 1, b1 = dg & 2;
+          const float m0 = (b0 ? o1 : o0) + __shfl_xor_sync(0xffffffffu, b0 ? o0 : o1, 1);
+          const float m1 = (b0 ? o3 : o2) + __shfl_xor_sync(0xffffffffu, b0 ? o2 : o3, 1);
+          const float sum = (b1 ? m1 : m0) + __shfl_xor_sync(0xffffffffu, b1 ? m0 : m1, 2);
+          if (col0 + dg < vdim) out[(size_t)(t0 + tt) * heads * vdim + (size_t)h * vdim + col0 + dg] = sum;
+        }
+      }
+    }
+    if (more) store(buf ^ 1);
+    __syncthreads();
+  }
+  if (MODE == 1 && blockIdx.z == 0) {      // thread tid has multiplied the decays of key tid % DREG at some of the tokens
+    float* keep = ws_keep + ((size_t)blockIdx.x * heads + h) * dim;
+    if (NT >= DREG) {
+      products[tid] = prod;
+      __syncthreads();
+      if (tid < DREG && tid < dim) {
+        float p = products[tid];
+        for (int i = tid + DREG; i < NT; i += DREG) p *= products[i];
+        keep[tid] = p;
+      }
+    } else {                                // fewer threads than keys: the staged decays are gone, the products come from alpha itself
+      for (int d = tid; d < dim; d += NT) {
+        float p = 1.0f;
+        for (int t = start; t < end; ++t) p *= alpha[(size_t)t * QK + h * dim + d];
+        keep[d] = p;
+      }
+    }
+  }
+  if (MODE == 2 && k != chunks_of_row - 1) return;
+  float* hd = MODE == 1 ? wsh : slot;                     // where the walk's end goes
+  if (!live) return;
+#pragma unroll
+  for (int i = 0; i < DG; ++i) {
+    const int d = 4 * i + dg;
+    if (d >= dim) continue;
+    float* dst = hd + (size_t)d * vdim + col0;
+    if (wide && col0 < vdim) {
+      *reinterpret_cast<float4*>(dst) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+        if (col0 + c < vdim) dst[c] = S[i][c];
+    }
+  }
+}
+
+// Heads of more than 128 keys: S in shared memory after the staging area, [dim][32]. The modes are those of gla_tile_kernel.
+template <typename T, int MODE>
 __global__ void __launch_bounds__(32) gla_scan_kernel(const T* u, int64_t ld, float q_scale, const float* alpha, GlaGate<T> gate,
                                                      float* out, float* state, int64_t state_stride, const int32_t* __restrict__ q_indptr,
                                                      const int32_t* __restrict__ slots, int rows, int heads, int dim, int vdim, float* ws, float* ws_keep) {
-  extern __shared__ float4 sm4[];    // two staging slots of dim (k, q, alpha, -); then S when it does not live in registers
-  constexpr int NREG = DREG > 0 ? DREG : 1;
-  constexpr int NN = DREG > 0 ? DREG / 32 : 32;          // entries of q, k and alpha a lane loads (dim <= 1024 in shared-memory form)
+  extern __shared__ float4 sm4[];    // two staging slots of dim (k, q, alpha, -); then S
+  constexpr int NN = 32;                                 // entries of q, k and alpha a lane loads (dim <= 1024)
   pdl_launch_dependents();
   int r = blockIdx.x, k = 0, chunks_of_row = 1;
   const int h = blockIdx.y, slice = blockIdx.z;
@@ -111,17 +274,11 @@ __global__ void __launch_bounds__(32) gla_scan_kernel(const T* u, int64_t ld, fl
   float* slot = state + (size_t)slots[r] * state_stride + (size_t)h * head_state;
   float* wsh = MODE != 0 ? ws + ((size_t)blockIdx.x * heads + h) * head_state : nullptr;
   const float* hs = MODE == 0 ? slot : wsh;               // where the walk starts from (MODE 1 starts empty)
-  float* S_sm = reinterpret_cast<float*>(sm4 + 2 * dim) + lane;      // [dim][32], used when DREG == 0
+  float* S = reinterpret_cast<float*>(sm4 + 2 * dim) + lane;      // [dim][32]
   const int QK = heads * dim;
   pdl_wait();
   if (end <= start) return;
-  float S[NREG];
-  if (DREG > 0) {
-#pragma unroll
-    for (int d = 0; d < NREG; ++d) S[d] = (MODE != 1 && live && d < dim) ? hs[(size_t)d * vdim + col] : 0.f;
-  } else {
-    for (int d = 0; d < dim; ++d) S_sm[(size_t)d * 32] = (MODE != 1 && live) ? hs[(size_t)d * vdim + col] : 0.f;
-  }
+  for (int d = 0; d < dim; ++d) S[(size_t)d * 32] = (MODE != 1 && live) ? hs[(size_t)d * vdim + col] : 0.f;
   // the next token's inputs, loaded one token ahead
   float nk[NN], nq[NN], na[NN], prod[NN], nv;
 #pragma unroll
@@ -160,22 +317,11 @@ __global__ void __launch_bounds__(32) gla_scan_kernel(const T* u, int64_t ld, fl
     if (t + 1 < end) load(t + 1);
     __syncwarp();
     float num = 0.f;
-    if (DREG > 0) {
-#pragma unroll
-      for (int d = 0; d < NREG; ++d) {
-        if (d < dim) {
-          const float4 f = stage[d];
-          S[d] = fmaf(f.z, S[d], f.x * val);
-          if (MODE != 1) num = fmaf(S[d], f.y, num);
-        }
-      }
-    } else {
-      for (int d = 0; d < dim; ++d) {
-        const float4 f = stage[d];
-        const float s = fmaf(f.z, S_sm[(size_t)d * 32], f.x * val);
-        S_sm[(size_t)d * 32] = s;
-        if (MODE != 1) num = fmaf(s, f.y, num);
-      }
+    for (int d = 0; d < dim; ++d) {
+      const float4 f = stage[d];
+      const float s = fmaf(f.z, S[(size_t)d * 32], f.x * val);
+      S[(size_t)d * 32] = s;
+      if (MODE != 1) num = fmaf(s, f.y, num);
     }
     if (MODE != 1 && live) out[(size_t)t * heads * vdim + (size_t)h * vdim + col] = num;
   }
@@ -189,15 +335,8 @@ __global__ void __launch_bounds__(32) gla_scan_kernel(const T* u, int64_t ld, fl
   }
   if (MODE == 2 && k != chunks_of_row - 1) return;
   float* hd = MODE == 1 ? wsh : slot;                     // where the walk's end goes
-  if (live) {
-    if (DREG > 0) {
-#pragma unroll
-      for (int d = 0; d < NREG; ++d)
-        if (d < dim) hd[(size_t)d * vdim + col] = S[d];
-    } else {
-      for (int d = 0; d < dim; ++d) hd[(size_t)d * vdim + col] = S_sm[(size_t)d * 32];
-    }
-  }
+  if (live)
+    for (int d = 0; d < dim; ++d) hd[(size_t)d * vdim + col] = S[(size_t)d * 32];
 }
 
 // One thread an entry of S of a (row, head): the row's state through its chunks in order. ws[chunk] holds the chunk's own S' on entry
@@ -243,32 +382,50 @@ static int gla_scan_launch(const T* u, int64_t ld, float q_scale, const float* a
                            const int32_t* q_indptr, const int32_t* slots, int rows, int tokens, int heads, int dim, int vdim, float* ws, float* ws_keep,
                            cudaStream_t s) {
   const int slices = (vdim + 31) / 32;
-  const size_t stage = (size_t)2 * dim * sizeof(float4);
   const int chunks = roost_gla_scan_chunks(tokens, rows);
-#define ROOST_GLA_LAUNCH(DREG, MODE, SMEM, GX)                                                                                              \
-  do {                                                                                                                                      \
-    auto kernel = gla_scan_kernel<T, DREG, MODE>;                                                                                           \
-    if ((SMEM) > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(SMEM));                         \
-    launch_kernel(kernel, dim3((GX), heads, slices), dim3(32), (SMEM), s, u, ld, q_scale, alpha, gate, out, state, state_stride, q_indptr,  \
-                  slots, rows, heads, dim, vdim, ws, ws_keep);                                                                              \
-  } while (0)
-#define ROOST_GLA_SCAN(DREG, SMEM)                                                                                                          \
+#define ROOST_GLA_THREE(LAUNCH)                                                                                                             \
   do {                                                                                                                                      \
     if (ws == nullptr) {                                                                                                                    \
-      ROOST_GLA_LAUNCH(DREG, 0, SMEM, rows);                                                                                                \
+      LAUNCH(0, rows);                                                                                                                      \
     } else {                                                                                                                                \
-      ROOST_GLA_LAUNCH(DREG, 1, SMEM, chunks);                                                                                              \
+      LAUNCH(1, chunks);                                                                                                                    \
       launch_kernel(gla_carry_kernel, dim3(rows, heads, (dim * vdim + 255) / 256), dim3(256), 0, s, (const float*)state, state_stride, ws,  \
                     (const float*)ws_keep, q_indptr, slots, heads, dim, vdim);                                                              \
-      ROOST_GLA_LAUNCH(DREG, 2, SMEM, chunks);                                                                                              \
+      LAUNCH(2, chunks);                                                                                                                    \
     }                                                                                                                                       \
   } while (0)
-  if (dim <= 32) ROOST_GLA_SCAN(32, stage);
-  else if (dim <= 64) ROOST_GLA_SCAN(64, stage);
-  else if (dim <= 128) ROOST_GLA_SCAN(128, stage);
-  else ROOST_GLA_SCAN(0, stage + (size_t)dim * 32 * sizeof(float));
-#undef ROOST_GLA_SCAN
-#undef ROOST_GLA_LAUNCH
+  auto tile = [&](auto dreg, auto warps) {
+    constexpr int D = decltype(dreg)::value, W = decltype(warps)::value;
+#define ROOST_GLA_TILE(MODE, GX)                                                                                                            \
+  launch_kernel(gla_tile_kernel<T, D, W, MODE>, dim3((GX), heads, (slices + W - 1) / W), dim3(32 * W), 0, s, u, ld, q_scale, alpha, gate,   \
+                out, state, state_stride, q_indptr, slots, rows, heads, dim, vdim, ws, ws_keep)
+    ROOST_GLA_THREE(ROOST_GLA_TILE);
+#undef ROOST_GLA_TILE
+  };
+  auto heads_of = [&](auto dreg) {
+    if (slices >= 3) tile(dreg, std::integral_constant<int, 4>());
+    else if (slices == 2) tile(dreg, std::integral_constant<int, 2>());
+    else tile(dreg, std::integral_constant<int, 1>());
+  };
+  if (dim <= 32) {
+    heads_of(std::integral_constant<int, 32>());
+  } else if (dim <= 64) {
+    heads_of(std::integral_constant<int, 64>());
+  } else if (dim <= 128) {
+    heads_of(std::integral_constant<int, 128>());
+  } else {
+    const size_t smem = (size_t)2 * dim * sizeof(float4) + (size_t)dim * 32 * sizeof(float);
+#define ROOST_GLA_WALK(MODE, GX)                                                                                                            \
+  do {                                                                                                                                      \
+    auto kernel = gla_scan_kernel<T, MODE>;                                                                                                 \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                             \
+    launch_kernel(kernel, dim3((GX), heads, slices), dim3(32), smem, s, u, ld, q_scale, alpha, gate, out, state, state_stride, q_indptr,    \
+                  slots, rows, heads, dim, vdim, ws, ws_keep);                                                                              \
+  } while (0)
+    ROOST_GLA_THREE(ROOST_GLA_WALK);
+#undef ROOST_GLA_WALK
+  }
+#undef ROOST_GLA_THREE
   return check_launch("gla_scan");
 }
 

@@ -104,8 +104,7 @@ class Run:
         worst, bound = (F32_TOKEN, F32_RMS) if self.dtype == torch.float32 else (BF16_TOKEN, BF16_RMS)
         keep = torch.ones(got.shape[0], dtype=torch.bool)
         if self.dtype != torch.float32 and bool((position_errors(got, want) >= worst).any()):
-            # A router whose two best logits lie closer than a rounding, or a norm that keeps only the direction of an output next to zero, moves
-            # a position's logits far for the smallest change. A position over the bound is ill-conditioned, not faulty, when rounding the plain
+            # A norm that keeps only the direction of an output next to zero moves a position's logits far for the smallest change. A position over the bound is ill-conditioned, not faulty, when rounding the plain
             # implementation's inputs and projections to 16 bits (as they are, and after a relative change of up to 2^-8) moves its logits far
             # by itself. Such positions are left out in 16 bits; the 32-bit run of the same kernels checks them.
             moved = position_errors(P.forward(self.cfg, weights, ids, rounding=lambda z: z.to(torch.bfloat16).double()), want)

@@ -219,7 +219,18 @@ def test_latent_attention_with_a_query_latent_neighbouring_pairs_and_sinks(kerne
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(4, 32, 64, 16, 16.0), (2, 6, 7, 3, 1.0), (1, 100, 33, 5, 4.0), (3, 128, 96, 16, 16.0), (1, 160, 40, 24, 8.0), (2, 64, 1, 1, 2.0)])
+@pytest.mark.parametrize("width,col", [(8, 0), (24, 16), (37, 3), (1024, 40), (4096, 8)])
+def test_a_gate_for_every_number_of_a_row(kernels, dtype, width, col):
+    g = torch.Generator().manual_seed(width)
+    T = 11
+    x, u = torch.randn(T, width, generator=g).to(dtype), (2.0 * torch.randn(T, col + width + 8, generator=g)).to(dtype)
+    got = kernels.head_gate_mul_(x.clone().cuda(), u.cuda(), col, width)
+    close(got.cpu(), x.double() * P.sigmoid(u[:, col : col + width].double()), dtype, "gate", f32=1e-6, bf16=1e-2)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(4, 32, 64, 16, 16.0), (2, 6, 7, 3, 1.0), (1, 100, 33, 5, 4.0), (3, 128, 96, 16, 16.0), (1, 160, 40, 24, 8.0), (2, 64, 1, 1, 2.0),
+                                                      (8, 64, 128, 16, 16.0), (2, 128, 20, 4, 16.0), (5, 20, 200, 9, 16.0)])
 @pytest.mark.parametrize("form", ["rows", "walk", "chunks"])
 def test_gated_linear_attention(kernels, dtype, heads, dim, vdim, rank, tau, form):
     g = torch.Generator().manual_seed(heads * dim + vdim)

@@ -1,7 +1,8 @@
 """Small Zufusun models for the tests: configurations that differ in every size and option, and weights drawn so that faults show.
 
 Weights: matrices N(0, std) scaled by their fan-in; norm weights around 1, those of the norms after sublayers around 0.7 so that a sublayer stays
-a little smaller than the stream. ``sharpen`` makes one query token of the first layer read one key token far above all others, so that
+a little smaller than the stream. Routers mostly read four elements of the stream that only the embedding fills (a token's class), under
+weights whose choice is clear for every class: rounding then never moves a token to another expert. ``sharpen`` makes one query token of the first layer read one key token far above all others, so that
 whether that key is seen decides the output.
 """
 from __future__ import annotations
@@ -51,11 +52,11 @@ MIXED = config([(latent(), moe()), (attention(), moe(experts=4, top=3, ff=20, li
 # decay rank of one, every expert chosen, two layers that read one latent, layers without a feed-forward, a gla layer first
 ODD = config([(gla(heads=1, dim=10, vdim=10, tau=1.0, decay_rank=1), None),
               (attention(heads=3, kv_heads=3, dim=10, vdim=10, scale=0.3, window=1, keep=1), moe(experts=3, top=3, ff=31, limit=0.3)),
-              (latent(heads=1, dim=4, rot_dim=2, vdim=9, q_rank=5, kv_rank=9, scale=1.1, base=10000.0), None),
+              (latent(heads=1, dim=4, rot_dim=2, vdim=9, q_rank=10, kv_rank=9, scale=0.6, base=10000.0), None),
               (latent(heads=6, dim=7, rot_dim=2, vdim=4, q_rank=13, kv_rank=9, scale=0.4, base=10000.0, kv_from=2), moe(experts=2, top=1, ff=10)),
               (attention(heads=6, kv_heads=2, dim=4, vdim=7, scale=1.1, window=40, keep=0), None),
-              (latent(heads=2, dim=4, rot_dim=2, vdim=3, q_rank=6, kv_rank=9, scale=0.7, base=10000.0, kv_from=2), None),
-              (gla(heads=4, dim=3, vdim=2, tau=30.0, decay_rank=5), moe(experts=6, top=2, ff=16, limit=50.0)),
+              (latent(heads=2, dim=4, rot_dim=2, vdim=10, q_rank=11, kv_rank=9, scale=0.5, base=10000.0, kv_from=2), None),
+              (gla(heads=3, dim=7, vdim=12, tau=30.0, decay_rank=5), moe(experts=6, top=2, ff=16, limit=50.0)),
               (attention(heads=2, kv_heads=1, dim=6, vdim=6, scale=0.6, window=3, keep=22), None)], width=36, vocab=61, eps=1e-6)
 # sizes of whole vectors (multiples of 8 and 64) that the tensor-core kernels serve, heads of more than 128 keys (the state in shared memory),
 # windows and kept keys at and beside the kernels' tiles, more query heads than a fragment has rows, experts of whole tiles
@@ -119,8 +120,30 @@ def draw_tensors(cfg, seed: int, std: float = 0.12) -> dict:
             t = 1.5 * r
         else:
             t = 2.0 * std * r * fan
+        if name.endswith("norm1") or name.endswith("norm2"):
+            t[CLASS_AT : CLASS_AT + CLASSES] = 0.0       # no sublayer writes a token's class
+        elif name == "embed":
+            t[:, CLASS_AT : CLASS_AT + CLASSES] = 2.0 * torch.nn.functional.one_hot(torch.randint(CLASSES, (shape[0],), generator=g), CLASSES)
+        elif name.endswith("mlp.router"):
+            t *= 0.1
+            t[:, CLASS_AT : CLASS_AT + CLASSES] = clear_choices(shape[0], cfg["layers"][int(name[1 : name.index(".")])]["mlp"]["router"]["top"], g)
         out[name] = t.to(torch.bfloat16)
     return out
+
+
+CLASS_AT, CLASSES = 2, 4
+
+
+def clear_choices(experts: int, top: int, g) -> torch.Tensor:
+    """[experts, classes]: of many draws the one whose last chosen and first unchosen logits lie furthest apart in the worst class."""
+    best, widest = None, -1.0
+    for _ in range(200):
+        w = 0.75 * torch.randn(experts, CLASSES, generator=g)
+        z = w.sort(dim=0, descending=True).values
+        gap = float((z[top - 1] - z[top]).min()) if top < experts else 1.0
+        if gap > widest:
+            best, widest = w, gap
+    return best
 
 
 def sharpen(cfg, tensors: dict, key_token: int, query_token: int, part: str, value: float = 6.0) -> None:
