@@ -92,7 +92,7 @@ class Paged:
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 8, 6), (3, 3, 20, 33), (6, 3, 96, 96), (8, 2, 64, 64), (5, 1, 16, 16), (4, 4, 128, 128), (32, 4, 128, 128),
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 8, 6), (3, 3, 20, 33), (6, 2, 80, 80), (8, 2, 64, 64), (5, 1, 16, 16), (4, 4, 128, 128), (32, 4, 128, 128),
                                                      (2, 1, 256, 256), (1, 1, 300, 40)])
 def test_the_attention_with_a_window_beside_the_first_keys(kernels, dtype, heads, kv_heads, dim, vdim):
     g = torch.Generator().manual_seed(heads * dim + vdim)
@@ -117,7 +117,7 @@ def test_the_attention_with_a_window_beside_the_first_keys(kernels, dtype, heads
     close(dev[:, :Q].cpu(), qn.reshape(T, Q), dtype, "normed queries in place", f32=2e-6, bf16=1e-2)      # ... and no slot: nothing cached
     group = heads // kv_heads
 
-    for window, keep in ((40, 7), (96, 20), (33, 64), (1, 1), (64, 0), (500, 30), (130, 100)):
+    for window, keep in ((40, 7), (90, 24), (33, 64), (1, 1), (64, 0), (500, 30), (130, 100)):
         want = torch.zeros(T, heads, vdim, dtype=torch.float64)
         for t in range(T):
             p, base = int(pg.positions[t]), t - int(pg.positions[t])
@@ -166,7 +166,7 @@ def test_the_attention_with_a_window_beside_the_first_keys(kernels, dtype, heads
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,nope,rope,rot,rank,q_rank", [(4, 64, 32, 32, 96, 128), (3, 10, 6, 4, 20, 7), (16, 128, 64, 64, 512, 384), (1, 8, 2, 2, 8, 1), (20, 16, 16, 16, 64, 40)])
+@pytest.mark.parametrize("heads,nope,rope,rot,rank,q_rank", [(5, 48, 32, 32, 80, 112), (3, 10, 6, 4, 20, 7), (16, 128, 64, 64, 512, 384), (1, 8, 2, 2, 8, 1), (20, 16, 16, 16, 64, 40)])
 def test_latent_attention_with_a_query_latent_neighbouring_pairs_and_sinks(kernels, dtype, heads, nope, rope, rot, rank, q_rank):
     g = torch.Generator().manual_seed(heads * rank)
     lens, page = [45, 203], 8
@@ -229,7 +229,7 @@ def test_a_gate_for_every_number_of_a_row(kernels, dtype, width, col):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(4, 32, 64, 16, 16.0), (2, 6, 7, 3, 1.0), (1, 100, 33, 5, 4.0), (3, 128, 96, 16, 16.0), (1, 160, 40, 24, 8.0), (2, 64, 1, 1, 2.0),
+@pytest.mark.parametrize("heads,dim,vdim,rank,tau", [(4, 32, 48, 12, 8.0), (2, 6, 7, 3, 1.0), (1, 100, 33, 5, 4.0), (3, 128, 96, 16, 16.0), (1, 160, 40, 24, 8.0), (2, 64, 1, 1, 2.0),
                                                       (8, 64, 128, 16, 16.0), (2, 128, 20, 4, 16.0), (5, 20, 200, 9, 16.0)])
 @pytest.mark.parametrize("form", ["rows", "walk", "chunks"])
 def test_gated_linear_attention(kernels, dtype, heads, dim, vdim, rank, tau, form):
